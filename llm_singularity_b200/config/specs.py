@@ -152,7 +152,12 @@ class KVAttentionSpec(PartSpec):
     loses ``2^(-8 (h + 1) / heads) * d``.  ``value_mix``: layers of one model that name the same
     ``value_mix_key`` share values within a token; the "source" layer (the first of them) caches its
     values as they are and lends them to the others for the step, a "mixed" layer caches
-    ``(1 - lambda) v + lambda v_source`` with its own learnt number ``vmix``."""
+    ``(1 - lambda) v + lambda v_source`` with its own learnt number ``vmix``.  ``diff``: differential
+    attention.  A head then has two queries and two keys of ``key_dim`` (stored and cached side by
+    side, [map 1, map 2]) over one value; with a_m the attention of map m, the head's output is
+    ``unit(a_1 - lambda a_2) * (1 - diff)``, ``unit`` the division by the root mean square over the
+    head (``eps``), and ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` one number of the layer
+    made of four learnt vectors of ``key_dim``.  It goes with position, window and chunk only."""
 
     hidden_size: int = 0
     num_heads: int = 0
@@ -177,6 +182,7 @@ class KVAttentionSpec(PartSpec):
     v_unit_norm: bool = False
     sink: bool = False
     gate_per_head: bool = False
+    diff: Optional[float] = None
     kind: str = field(init=False, default="kv_attention")
 
 
@@ -326,8 +332,8 @@ class GatedMLPSpec(PartSpec):
 class DenseMLPSpec(PartSpec):
     """down( act(up(x)) ), dense, no gate and no bias.  ``activation`` "bent_square" is a two-branch
     activation with two learnt numbers p and q stored with the layer: ``softplus(p) z^2 + z/2`` for
-    z > 0 and ``(1/2 + softplus(q)) (e^z - 1 - z) + z/2`` for z <= 0; "silu", "gelu_tanh" and "none"
-    need no parameter."""
+    z > 0 and ``(1/2 + softplus(q)) (e^z - 1 - z) + z/2`` for z <= 0; "silu", "gelu_tanh", "relu_squared"
+    (``max(z, 0)^2``) and "none" need no parameter."""
 
     hidden_size: int = 0
     intermediate_size: int = 0
@@ -337,16 +343,19 @@ class DenseMLPSpec(PartSpec):
 
 @dataclass(frozen=True)
 class MoESpec(PartSpec):
-    """Routed gated experts, no bias: ``sum over the chosen e of down_e(act(gate_e u) * up_e u)``.
+    """Routed experts, no bias: ``sum over the chosen e of down_e(act(gate_e u) * up_e u)``, or without
+    ``gated`` of ``down_e(act(up_e u))``.
 
-    Router logits are 32-bit; ``score`` turns them into scores ("sigmoid", or "softmax" over all
-    experts); the ``top`` largest are chosen; ``renormalize`` divides the chosen scores by their
+    Router logits are 32-bit (``router_bias``: with a learnt number per expert added); ``score`` turns them
+    into scores ("sigmoid", "softmax" over all experts, or "softmax_chosen" over the chosen logits
+    alone); the ``top`` largest are chosen; ``renormalize`` divides the chosen scores by their
     sum.  ``weight_on`` says what a score multiplies: the expert's "input" (``u = s x``) or its
     "output".  ``choice_bias``: a learnt number per expert is added to the scores for the choice only
     (the weights are the scores without it).  The chosen scores are divided by their sum +
     ``renorm_eps`` and multiplied by ``weight_scale``.  ``limit`` belongs to the activation
-    "capped_glu" (see ``GatedMLPSpec``).  ``shared``: a gated feed-forward that every token passes
-    besides its chosen experts; its result is added."""
+    "capped_glu" (see ``GatedMLPSpec``).  ``shared``: a feed-forward that every token passes
+    besides its chosen experts; its result is added, multiplied by sigmoid(W_sg x), one number per token,
+    with ``shared_gate``."""
 
     hidden_size: int = 0
     expert_size: int = 0
@@ -360,7 +369,10 @@ class MoESpec(PartSpec):
     weight_scale: float = 1.0
     renorm_eps: float = 0.0
     limit: float = 0.0
-    shared: Optional[GatedMLPSpec] = None
+    shared: Optional[PartSpec] = None
+    gated: bool = True
+    router_bias: bool = False
+    shared_gate: bool = False
     kind: str = field(init=False, default="moe")
 
 
@@ -390,6 +402,17 @@ class BlockSpec(PartSpec):
     mixer_norm: PartSpec = None
     ffn_norm: Optional[PartSpec] = None
     kind: str = field(init=False, default="pre_norm")
+
+
+@dataclass(frozen=True)
+class SideBySideBlockSpec(PartSpec):
+    """h = norm(x); x += mixer(h) + ffn(h)   (the "side_by_side" arrangement: one norm, both sublayers read
+    its output).  ``ffn`` None: the mixer alone."""
+
+    mixer: PartSpec = None
+    ffn: Optional[PartSpec] = None
+    norm: PartSpec = None
+    kind: str = field(init=False, default="side_by_side")
 
 
 @dataclass(frozen=True)

@@ -59,12 +59,17 @@ LSB_API int lsb_gated_act(const void* gate_up, void* out, int dtype, int tokens,
 // two-branch activation with two learnt numbers handed in already transformed: right of zero a
 // parabola, c_pos z^2 + z / 2; left of it a saturating branch, c_neg (e^z - 1 - z) + z / 2
 // (c_pos = softplus(p), c_neg = 1/2 + softplus(q) for the stored p and q).
-enum : int { LSB_ACT_BENT_SQUARE = 4 };
+// LSB_ACT_RELU_SQUARED: max(z, 0)^2.
+enum : int { LSB_ACT_BENT_SQUARE = 4, LSB_ACT_RELU_SQUARED = 6 };
 
 __device__ __forceinline__ float plain_act_of(float z, int act, float c_pos, float c_neg) {
     if (act == LSB_ACT_SILU) return z / (1.f + expf(-z));
     if (act == LSB_ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608f * (z + 0.044715f * z * z * z)));
     if (act == LSB_ACT_BENT_SQUARE) return z > 0.f ? c_pos * z * z + 0.5f * z : c_neg * (expm1f(z) - z) + 0.5f * z;
+    if (act == LSB_ACT_RELU_SQUARED) {
+        z = fmaxf(z, 0.f);
+        return z * z;
+    }
     return z;
 }
 
@@ -94,7 +99,7 @@ __global__ void plain_act_kernel(const T* __restrict__ x, T* __restrict__ out, l
 LSB_API int lsb_plain_act(const void* x, void* out, int dtype, long long total, int act, float c_pos, float c_neg,
                           cudaStream_t stream) {
     if (total <= 0) return 0;
-    if (act < LSB_ACT_SILU || act > LSB_ACT_BENT_SQUARE) return (int)cudaErrorInvalidValue;
+    if ((act < LSB_ACT_SILU || act > LSB_ACT_BENT_SQUARE) && act != LSB_ACT_RELU_SQUARED) return (int)cudaErrorInvalidValue;
     const int threads = 256;
     const int per = dtype == LSB_F32 ? 4 : 8;    // values in 16 bytes
     const int wide = total % 8 == 0 && ((reinterpret_cast<size_t>(x) | reinterpret_cast<size_t>(out)) & 15) == 0;

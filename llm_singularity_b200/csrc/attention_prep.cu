@@ -15,6 +15,10 @@
 //   * queries go to q_out [tokens, nh * dk]; keys and values to the token's place in the cache
 //     pages, [page][kv head][offset][dk] and [page][kv head][offset][dv].
 //
+// `maps` > 1: every query and key head is that many parts of dk side by side, each normed and rotated as
+// a head of its own (attention whose heads have several queries and keys over one value); a cached key
+// is then a row of maps * dk.
+//
 // Each of the first four is optional.  The projections come as rows of one matrix, q at q_off, k
 // at k_off, v at v_off, in the compute dtype.  One block per token: all its query and key channels
 // are brought into shared memory in one sweep, then a warp works on a head at a time; a token's
@@ -28,7 +32,7 @@ constexpr int kPrepMaxDim = 512;
 
 struct PrepArgs {
     const void* proj; long long ld; int q_off, k_off, v_off;
-    int nh, nkv, dk, dv;
+    int nh, nkv, dk, dv, maps;
     const float *q_bias, *k_bias, *v_bias;
     const float *q_norm, *k_norm; float norm_eps;
     int norm_all, v_unit;
@@ -63,7 +67,7 @@ template <> struct PrepVec<__nv_bfloat16> {
 
 template <typename T>
 __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArgs a) {
-    extern __shared__ float all_sh[];                   // [(nh + nkv) * dk]
+    extern __shared__ float all_sh[];                   // [(nh + nkv) * maps * dk]
     __shared__ float cs_sh[2][kPrepMaxDim / 2];
     __shared__ float sum_sh[33];
     lsb_pdl_launch_dependents();
@@ -82,7 +86,8 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
     // the first of the token's query and key channels are asked for before the block table is, so that
     // the two latencies pass together
     const T* row = (const T*)a.proj + (size_t)t * a.ld;
-    const int nq = a.nh * a.dk, nall = nq + a.nkv * a.dk;
+    const int nh = a.nh * a.maps, nkv = a.nkv * a.maps;     // parts of heads
+    const int nq = nh * a.dk, nall = nq + nkv * a.dk;
     constexpr int kAhead = 4, VEC = PrepVec<T>::N;
     T ahead[kAhead];
     uint4 ahead_v[2];
@@ -108,7 +113,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
             if (threadIdx.x == 0) lsb_set_status(LSB_BAD_PAGE);
         } else {
             const long long at = (long long)page * a.nkv * a.page_size + (pos % a.page_size);
-            k_base = at * a.dk;
+            k_base = at * a.maps * a.dk;
             v_base = at * a.dv;
         }
     }
@@ -165,9 +170,9 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
         inv_all_q = rsqrtf(lsb_block_sum(sq, sum_sh) / (float)nq + a.norm_eps);
         inv_all_k = rsqrtf(lsb_block_sum(sk, sum_sh) / (float)(nall - nq) + a.norm_eps);
     }
-    for (int head = warp; head < a.nh + a.nkv; head += kPrepWarps) {
-        const bool is_q = head < a.nh;
-        const int hh = is_q ? head : head - a.nh;
+    for (int head = warp; head < nh + nkv; head += kPrepWarps) {
+        const bool is_q = head < nh;
+        const int hh = is_q ? head : head - nh;
         const float* hs = all_sh + (size_t)head * a.dk;
         const float* nw = is_q ? a.q_norm : a.k_norm;
         if (nw && a.norm_all) nw += (size_t)hh * a.dk;
@@ -181,8 +186,11 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
         }
         const float mul = is_q ? temp : 1.f;
         T* dst = nullptr;
-        if (is_q) dst = (T*)a.q_out + ((size_t)t * a.nh + hh) * a.dk;
-        else if (k_base >= 0) dst = (T*)a.k_pages + k_base + (long long)hh * a.page_size * a.dk;
+        if (is_q) dst = (T*)a.q_out + ((size_t)t * nh + hh) * a.dk;
+        else if (k_base >= 0) {
+            const int kv = a.maps == 1 ? hh : hh / a.maps;
+            dst = (T*)a.k_pages + k_base + (long long)kv * a.page_size * a.maps * a.dk + (hh - kv * a.maps) * a.dk;
+        }
         if (dst) {
             // work items: pairs of dims; the rotating pairs first, then the rest two by two
             const int pairs = (a.dk + 1) >> 1;
@@ -256,18 +264,18 @@ LSB_API int lsb_attention_prep_max_dim() { return kPrepMaxDim; }
 LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_off, int k_off, int v_off, int tokens,
                                int nh, int nkv, int dk, int dv, const float* q_bias, const float* k_bias,
                                const float* v_bias, const float* q_norm, const float* k_norm, float norm_eps,
-                               int norm_all, int v_unit, float temp_coef, int temp_every, const float* inv_freq, int rotary_dim, int adjacent,
+                               int norm_all, int v_unit, int maps, float temp_coef, int temp_every, const float* inv_freq, int rotary_dim, int adjacent,
                                const int* positions, const int* token_req, const int* table_rows,
                                const int* block_table, int table_stride, void* q_out, void* k_pages, void* v_pages,
                                int page_size, int num_pages, int store, const void* v_first, long long v_first_ld,
                                const float* v_lambda, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (dk <= 0 || dk > kPrepMaxDim || dv <= 0 || nh <= 0 || nkv <= 0 || rotary_dim % 2 || rotary_dim > dk ||
+    if (dk <= 0 || dk > kPrepMaxDim || maps < 1 || dv <= 0 || nh <= 0 || nkv <= 0 || rotary_dim % 2 || rotary_dim > dk ||
         rotary_dim < 0 || (rotary_dim > 0 && !inv_freq) || (v_first && (!v_lambda || v_unit)))
         return (int)cudaErrorInvalidValue;
     PrepArgs a;
     a.proj = proj; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
-    a.nh = nh; a.nkv = nkv; a.dk = dk; a.dv = dv;
+    a.nh = nh; a.nkv = nkv; a.dk = dk; a.dv = dv; a.maps = maps;
     a.q_bias = q_bias; a.k_bias = k_bias; a.v_bias = v_bias;
     a.q_norm = q_norm; a.k_norm = k_norm; a.norm_eps = norm_eps;
     a.norm_all = norm_all; a.v_unit = v_unit;
@@ -281,7 +289,7 @@ LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_
     const int per16 = dtype == LSB_F32 ? 4 : 8;
     a.vec = ((uintptr_t)proj % 16 == 0 && (uintptr_t)v_pages % 16 == 0 && ld % per16 == 0 && q_off % per16 == 0 &&
              k_off % per16 == 0 && v_off % per16 == 0 && dk % per16 == 0 && dv % per16 == 0) ? 1 : 0;
-    const size_t smem = (size_t)(nh + nkv) * dk * sizeof(float);
+    const size_t smem = (size_t)(nh + nkv) * maps * dk * sizeof(float);
     if (smem > 160 * 1024) return (int)cudaErrorInvalidValue;
     LSB_DISPATCH_DTYPE(dtype, {
         if (smem > 32 * 1024) {

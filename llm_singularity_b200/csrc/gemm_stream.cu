@@ -30,6 +30,8 @@
 //
 // act != 0: w has 2 * N_out rows alternating gate_i, up_i and out is [M, N / 2] with
 // out[m, i] = act(d[m, 2i]) * d[m, 2i + 1] (1 silu, 2 gelu in its tanh form, 3 none), in 32-bit.
+// act = LSB_PLAIN + an id: an ungated product with that activation on every element (1, 2, or 6 for the
+// square of relu).
 //
 // The reference calls cublasSgemm for every projection (kernels/src/cublas_provider.cpp:36-51) and
 // a separate kernel for silu(g) * u (kernels/src/activations.cu:11-21).  No load here uses cluster
@@ -62,6 +64,7 @@ struct StreamParams {
     int M, N, K;
     int out_f32;
     int act;            // 0: plain product; else the activation of a gated product
+    int plain;          // the activation of an ungated product (0: none)
     float limit;        // the cap of LSB_ACT_CAPPED_GLU: min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1)
     int kc;             // K per stage (a multiple of 128)
     int stages;
@@ -147,6 +150,14 @@ __device__ __forceinline__ float gate_act(float g, int act) {
     if (act == LSB_ACT_SILU) return g / (1.f + __expf(-g));
     if (act == LSB_ACT_GELU_TANH) return 0.5f * g * (1.f + tanhf(0.7978845608f * (g + 0.044715f * g * g * g)));
     return g;
+}
+enum : int { LSB_ACT_RELU_SQUARED = 6, LSB_PLAIN = 16 };
+__device__ __forceinline__ float plain_act(float z, int act) {
+    if (act == LSB_ACT_RELU_SQUARED) {
+        z = fmaxf(z, 0.f);
+        return z * z;
+    }
+    return gate_act(z, act);
 }
 __device__ __forceinline__ float gate_times_up(float g, float u, int act, float limit) {
     if (act == LSB_ACT_CAPPED_GLU) {
@@ -294,13 +305,13 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
     // parameter read for the first time costs a trip past the constant cache (some 0.3 us each,
     // one after the other, in a kernel whose whole end is 1 us), and here it hides under the wait
     // for the first weights.
-    int e_M = prm.M, e_N = prm.N, e_act = prm.act, e_f32 = prm.out_f32;
+    int e_M = prm.M, e_N = prm.N, e_act = prm.act, e_f32 = prm.out_f32, e_plain = prm.plain;
     void* e_out = prm.out;
     float e_inv = prm.inv_size, e_eps = prm.eps, e_limit = prm.limit;
     float* e_res = prm.residual;
     const float* e_nw = prm.norm_w;
     float* e_ss = prm.ss_out;
-    asm volatile("" : "+r"(e_M), "+r"(e_N), "+r"(e_act), "+r"(e_f32), "+l"(e_out), "+f"(e_inv), "+f"(e_eps), "+f"(e_limit),
+    asm volatile("" : "+r"(e_M), "+r"(e_N), "+r"(e_act), "+r"(e_f32), "+r"(e_plain), "+l"(e_out), "+f"(e_inv), "+f"(e_eps), "+f"(e_limit),
                       "+l"(e_res), "+l"(e_nw), "+l"(e_ss));
     const int n_out = e_act ? e_N / 2 : e_N;
     const int k_steps = kc >> 4;               // a multiple of kInFlight (beyond K the copy has filled in zeros)
@@ -409,6 +420,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                 v = 0.f;
                 for (int p = 0; p < parts; ++p) v += src[(size_t)p * part_stride];
                 v *= scale;
+                if (e_plain) v = plain_act(v, e_plain);
             }
             const size_t o = (size_t)m * n_out + first + j;
             if (ADDS) {
@@ -534,6 +546,7 @@ static int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int box_
 
 LSB_API int lsb_gemm_stream_supported(const void* x, const void* w, int M, int N, int K, int act) {
     Plan p;
+    if (act >= LSB_PLAIN) act = 0;
     return ((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0 && make_plan(M, N, K, act, 1, sm_count(), &p) &&
            get_encode() != nullptr;
 }
@@ -541,6 +554,7 @@ LSB_API int lsb_gemm_stream_supported(const void* x, const void* w, int M, int N
 // The number of blocks a product of these sizes runs with: the parts its sums of squares come in.
 LSB_API int lsb_gemm_stream_blocks(int M, int N, int K, int act) {
     Plan p;
+    if (act >= LSB_PLAIN) act = 0;
     return make_plan(M, N, K, act, 1, sm_count(), &p) ? p.blocks : 0;
 }
 
@@ -576,6 +590,10 @@ static int stream_product(const void* x, const void* w, void* out, int out_f32, 
                           float* residual, const float* norm_w, float* ss_out, const void* warm,
                           cudaStream_t stream) {
     Plan p;
+    const int plain = act >= LSB_PLAIN ? act - LSB_PLAIN : 0;
+    if (plain) act = 0;
+    if (plain && (residual || (plain != LSB_ACT_SILU && plain != LSB_ACT_GELU_TANH && plain != LSB_ACT_RELU_SQUARED)))
+        return (int)cudaErrorInvalidValue;
     if (act == LSB_ACT_CAPPED_GLU && !(limit > 0.f)) return (int)cudaErrorInvalidValue;
     if (!lsb_gemm_stream_supported(x, w, M, N, K, act)) return (int)cudaErrorInvalidValue;
     if (ss_in && (ss_parts <= 0 || ss_parts > 32 * kSsPerLane || size <= 0)) return (int)cudaErrorInvalidValue;
@@ -584,7 +602,7 @@ static int stream_product(const void* x, const void* w, void* out, int out_f32, 
     StreamParams prm;
     prm.x = (const bf16*)x; prm.w = (const bf16*)w; prm.out = out;
     prm.M = M; prm.N = N; prm.K = K;
-    prm.out_f32 = out_f32; prm.act = act; prm.limit = limit;
+    prm.out_f32 = out_f32; prm.act = act; prm.limit = limit; prm.plain = plain;
     prm.kc = p.kc; prm.stages = p.stages; prm.unit = p.unit; prm.w_bytes = p.w_bytes;
     prm.rows_a = p.rows_a; prm.rows_b = p.rows_b; prm.rows_c = p.rows_c;
     prm.rt = p.rt;

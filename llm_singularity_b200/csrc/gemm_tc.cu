@@ -153,6 +153,7 @@ struct GemmParams {
     int act;                      // gated products: 1 silu, 2 gelu (tanh form), 3 none (gate * up), 5 capped
     float limit;                  // ... whose cap this is
                                   // The output then has half as many columns: silu(gate) * up.
+    int plain;                    // ungated products: the activation on every element (0: none)
     int static_operand;           // 1: P holds weights, 2: Q does (loaded before the PDL wait)
     void* out;                    // bf16 or float
     // Grouped products (routed experts): Q stacks one matrix of `group_rows` rows per group, and
@@ -192,6 +193,21 @@ __device__ __forceinline__ float gate_mul(float g, float u, int act, float limit
     }
     const float a = act == LSB_ACT_GELU_TANH ? 1.5957691216f * (g + 0.044715f * g * g * g) : g;
     return __fdividef(g, 1.f + __expf(-a)) * u;
+}
+// The activation of an ungated product, by the ids above plus the square of relu; the caller adds
+// LSB_PLAIN to the id to say that the product is ungated.
+enum : int { LSB_ACT_RELU_SQUARED = 6, LSB_PLAIN = 16 };
+__device__ __forceinline__ float plain_act(float z, int act) {
+    if (act == LSB_ACT_RELU_SQUARED) {
+        z = fmaxf(z, 0.f);
+        return z * z;
+    }
+    const float a = act == LSB_ACT_GELU_TANH ? 1.5957691216f * (z + 0.044715f * z * z * z) : z;
+    return __fdividef(z, 1.f + __expf(-a));
+}
+__device__ __forceinline__ void plain_act_all(uint32_t (&r)[32], int act) {
+#pragma unroll
+    for (int x = 0; x < 32; ++x) r[x] = __float_as_uint(plain_act(__uint_as_float(r[x]), act));
 }
 #define silu_mul(g, u) gate_mul((g), (u), prm.act, prm.limit)
 
@@ -249,6 +265,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& prm, uint32_t (&r)
         }
         return;
     }
+    if (prm.plain) plain_act_all(r, prm.plain);
     const long long o = (long long)i * prm.ldc_i + (long long)j * prm.ldc_j;
     if (prm.out_f32) {
         float* dst = reinterpret_cast<float*>(prm.out) + o;
@@ -311,6 +328,7 @@ __device__ __forceinline__ void epilogue_staged(const GemmParams& prm, unsigned 
                 mine[lane * CPROW + (cc ^ (lane & 7))] = make_uint4(w[0], w[1], w[2], w[3]);
             }
         } else {
+            if (prm.plain) plain_act_all(r, prm.plain);
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
                 uint32_t w[4];
@@ -559,6 +577,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
 #pragma unroll
                 for (int peer = 0; peer < 8; ++peer)          // summed in rank order
                     if (peer < prm.splits) { acc.x += v[peer].x; acc.y += v[peer].y; acc.z += v[peer].z; acc.w += v[peer].w; }
+                if (prm.plain) {
+                    acc.x = plain_act(acc.x, prm.plain); acc.y = plain_act(acc.y, prm.plain);
+                    acc.z = plain_act(acc.z, prm.plain); acc.w = plain_act(acc.w, prm.plain);
+                }
                 const int i = i0 + row, j = j0 + c4 * 4;
                 if (i < prm.rows_p) {
                     const long long o0 = (long long)i * prm.ldc_i + (long long)j * prm.ldc_j;
@@ -943,14 +965,18 @@ LSB_API int lsb_gemm_tc_plan(int M, int N, int K, int swiglu, int* swap, int* bn
 // out[M, N] = x[M, K] * w[N, K]^T, bf16 inputs, bf16 or float output.
 // swiglu != 0: w has 2 * N_out rows alternating gate_i, up_i; out is [M, N / 2] with
 // out[m, i] = act(d[m, 2i]) * d[m, 2i + 1], act named by swiglu: 1 silu, 2 gelu (tanh form), 3 none, 5 capped
-// (with its limit).
+// (with its limit).  swiglu = LSB_PLAIN + an id: an ungated product with that activation on every element
+// (silu, gelu in its tanh form, or the square of relu).
 static bool known_act(int act) { return (act >= 0 && act <= LSB_ACT_NONE) || act == LSB_ACT_CAPPED_GLU; }
+static bool known_plain(int act) { return act == LSB_ACT_SILU || act == LSB_ACT_GELU_TANH || act == LSB_ACT_RELU_SQUARED; }
 
 LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, int M, int N, int K,
                         int swiglu, float limit, cudaStream_t stream) {
+    const int plain = swiglu >= LSB_PLAIN ? swiglu - LSB_PLAIN : 0;
+    if (plain) swiglu = 0;
     if (!lsb_gemm_tc_supported(x, w, M, N, K)) return (int)cudaErrorInvalidValue;
     if (swiglu && (N % 2)) return (int)cudaErrorInvalidValue;
-    if (!known_act(swiglu)) return (int)cudaErrorInvalidValue;
+    if (!known_act(swiglu) || (plain && !known_plain(plain))) return (int)cudaErrorInvalidValue;
     int swap, bn, splits;
     lsb_gemm_tc_plan(M, N, K, swiglu, &swap, &bn, &splits);
     const int n_out = swiglu ? N / 2 : N;
@@ -963,6 +989,7 @@ LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, in
     prm.out = out;
     prm.act = swiglu;
     prm.limit = limit;
+    prm.plain = plain;
     prm.tile_group = nullptr;
     prm.group_rows = 0;
     const int sms = num_sms();
@@ -1048,10 +1075,13 @@ LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, in
 
 // Grouped form for routed experts: x [M, K] holds row tiles of 128 that belong to one group each
 // (tile_group[M / 128], device memory, -1 for an unused tile), w stacks `groups` matrices [N, K];
-// out[m] = x[m] w[group of m's tile]^T, gated as above if swiglu.  M is a multiple of 128.
+// out[m] = x[m] w[group of m's tile]^T, gated (or with a plain activation) as above if swiglu.  M is a multiple of 128.
 LSB_API int lsb_gemm_tc_grouped(const void* x, const void* w, void* out, int out_f32, int M, int N, int K,
                                 int groups, const int* tile_group, int swiglu, float limit, cudaStream_t stream) {
     if (M <= 0) return 0;
+    const int plain = swiglu >= LSB_PLAIN ? swiglu - LSB_PLAIN : 0;
+    if (plain) swiglu = 0;
+    if (plain && !known_plain(plain)) return (int)cudaErrorInvalidValue;
     if (!lsb_gemm_tc_supported(x, w, M, N, K) || M % kBM || groups <= 0 || !tile_group) return (int)cudaErrorInvalidValue;
     if ((swiglu && (N % 2)) || !known_act(swiglu)) return (int)cudaErrorInvalidValue;
     if ((long long)groups * N > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
@@ -1065,6 +1095,7 @@ LSB_API int lsb_gemm_tc_grouped(const void* x, const void* w, void* out, int out
     prm.out = out;
     prm.act = swiglu;
     prm.limit = limit;
+    prm.plain = plain;
     prm.tile_group = tile_group;
     prm.group_rows = N;
     prm.rows_p = M; prm.rows_q = N; prm.ldc_i = n_out; prm.ldc_j = 1;

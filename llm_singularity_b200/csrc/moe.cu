@@ -1,17 +1,18 @@
 // Routed experts: choosing, sorting rows by expert, the two grouped products and the sum.
 //
-//   moe_route    per token: scores from the 32-bit router logits (sigmoid, or softmax over all
-//                experts), the `top` largest (the lower index wins a tie), optionally divided by
-//                their sum -> ids [T, top], weights [T, top].
+//   moe_route    per token: scores from the 32-bit router logits (sigmoid, softmax over all experts,
+//                or softmax over the chosen alone), the `top` largest (the lower index wins a tie),
+//                optionally divided by their sum -> ids [T, top], weights [T, top].
 //   moe_align    the (token, choice) pairs sorted by expert into rows; each expert's rows start
 //                on a multiple of the row tile, so a tile of rows belongs to one expert.  Writes
 //                pos [T * top] (the row of each pair), row_token / row_scale [capacity] (-1 / 0 in
 //                the padding) and tile_expert [capacity / tile] (-1 beyond the last used tile).
 //   moe_up       rows gathered from x (times the row's weight if the weight goes on the input),
-//                times the expert's gate/up matrix (rows alternate gate_i, up_i), act(g) * u.
+//                times the expert's gate/up matrix (rows alternate gate_i, up_i), act(g) * u; or
+//                times its up matrix alone, act(u).
 //   moe_down     times the expert's down matrix -> y [capacity, hidden] 32-bit.
 //   moe_combine  out[t] = sum over the token's choices of y[pos] (times the weight if it goes on
-//                the output), rounded to T once.
+//                the output), plus a shared expert's row (times a sigmoid), rounded to T once.
 //
 // Each output row depends only on its own input row and its expert's weights, and the sum runs
 // over a token's choices in their order, so where a row landed does not change any result.
@@ -35,13 +36,24 @@ __device__ __forceinline__ float moe_gate_mul(float z, float up, int act, float 
     return z * up;
 }
 
-// How scores are made and weighted: `score` 0 sigmoid, 1 softmax over all experts; `bias` (one number an
-// expert, may be null) is added to the scores for the choice only; the chosen scores are divided by
-// their sum + eps if `renorm`, and multiplied by `scale`.
+// The activation of an ungated expert: 1 silu, 2 gelu in its tanh form, 6 the square of relu, else none.
+__device__ __forceinline__ float moe_plain(float z, int act) {
+    if (act == 6) {
+        z = fmaxf(z, 0.f);
+        return z * z;
+    }
+    return moe_gate_mul(z, 1.f, act, 0.f);
+}
+
+// How scores are made and weighted: `score` 0 sigmoid, 1 softmax over all experts, 2 softmax over the chosen
+// logits alone; `bias` (one number an expert, may be null) is added to the scores for the choice only, or,
+// with `joins`, to the logits themselves; the chosen scores are divided by their sum + eps if `renorm`,
+// and multiplied by `scale`.  A token's logits are `ld` numbers apart.
 struct RouteOpts {
     int score, renorm;
     const float* bias;
     float scale, eps;
+    int joins, ld;
 };
 
 constexpr int kMaxTop = 32;
@@ -50,12 +62,15 @@ constexpr int kMaxTop = 32;
 __device__ __forceinline__ void route_token(const float* __restrict__ z, int E, int top, const RouteOpts ro,
                                             int* __restrict__ ids, float* __restrict__ wts, int lane) {
     const int score = ro.score, renorm = ro.renorm;
+    const float* add = ro.joins ? ro.bias : nullptr;         // part of the logits
+    const float* correct = ro.joins ? nullptr : ro.bias;     // for the choice alone
+    auto logit = [&](int e) { return add ? z[e] + add[e] : z[e]; };
     float zmax = -FLT_MAX, denom = 1.f;
     if (score == 1) {
-        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
+        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, logit(e));
         zmax = lsb_warp_max(zmax);
         float s = 0.f;
-        for (int e = lane; e < E; e += 32) s += expf(z[e] - zmax);
+        for (int e = lane; e < E; e += 32) s += expf(logit(e) - zmax);
         denom = lsb_warp_sum(s);
     }
     int chosen[kMaxTop];
@@ -68,7 +83,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int E, 
             bool taken = false;
             for (int j = 0; j < k; ++j) taken |= (chosen[j] == e);
             // (without a bias the logits order the experts as their scores do)
-            const float c = ro.bias ? (score == 1 ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e]))) + ro.bias[e] : z[e];
+            const float c = correct ? (score == 1 ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e]))) + correct[e] : logit(e);
             if (!taken && (c > best || (c == best && e < bi))) { best = c; bi = e; }
         }
 #pragma unroll
@@ -78,14 +93,17 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int E, 
             if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
         }
         chosen[k] = bi;
-        if (ro.bias) best = z[bi];
-        val[k] = score == 1 ? expf(best - zmax) / denom : 1.f / (1.f + expf(-best));
+        if (correct) best = z[bi];
+        if (score == 2) {                   // (the first chosen is the largest)
+            if (k == 0) zmax = best;
+            val[k] = expf(best - zmax);
+        } else val[k] = score == 1 ? expf(best - zmax) / denom : 1.f / (1.f + expf(-best));
         total += val[k];
     }
     if (lane == 0) {
         for (int k = 0; k < top; ++k) {
             ids[k] = chosen[k];
-            wts[k] = (renorm ? val[k] / (total + ro.eps) : val[k]) * ro.scale;
+            wts[k] = (score == 2 ? val[k] / total : renorm ? val[k] / (total + ro.eps) : val[k]) * ro.scale;
         }
     }
 }
@@ -96,7 +114,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int n_tokens,
     lsb_pdl_wait();
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
     if (warp >= n_tokens) return;
-    route_token(logits + (size_t)warp * E, E, top, ro, ids + (size_t)warp * top, wts + (size_t)warp * top, lane);
+    route_token(logits + (size_t)warp * ro.ld, E, top, ro, ids + (size_t)warp * top, wts + (size_t)warp * top, lane);
 }
 
 __global__ void __launch_bounds__(1024)
@@ -111,7 +129,7 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
     lsb_pdl_wait();
     if (logits) {                       // a step of few tokens: the choosing is done here too, a warp a token
         for (int t = threadIdx.x >> 5; t < n / top; t += blockDim.x >> 5)
-            route_token(logits + (size_t)t * E, E, top, ro, ids + (size_t)t * top, wts + (size_t)t * top,
+            route_token(logits + (size_t)t * ro.ld, E, top, ro, ids + (size_t)t * top, wts + (size_t)t * top,
                         threadIdx.x & 31);
         __syncthreads();
     }
@@ -147,6 +165,7 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
 
 // MODE 0 (up):   A row = T(scale * x[row_token]) (scale 1 unless on_input), B = w[e] [2F, K], gated
 //                epilogue -> out T [capacity, F]
+// MODE 2 (up, ungated): as MODE 0 with B = w[e] [N, K] and a plain activation -> out T [capacity, N]
 // MODE 1 (down): A = h [capacity, K] T, B = w[e] [N, K] -> out 32-bit [capacity, N]
 template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
@@ -175,7 +194,7 @@ moe_gemm_kernel(const T* __restrict__ A, const int* __restrict__ row_token,
             const int k = k0 + tx, n = n0 + i;
             float a = 0.f;
             if (k < K && tok_sh[i] >= 0) {
-                if (MODE == 0)
+                if (MODE != 1)
                     a = lsb_to_float(lsb_from_float<T>(scale_sh[i] * lsb_to_float(A[(size_t)tok_sh[i] * K + k])));
                 else
                     a = lsb_to_float(A[(size_t)(m0 + i) * K + k]);
@@ -200,6 +219,8 @@ moe_gemm_kernel(const T* __restrict__ A, const int* __restrict__ row_token,
             const float up = __shfl_down_sync(0xffffffffu, acc[j], 1);
             if (!(tx & 1) && n + 1 < N)
                 ((T*)out_)[(size_t)m * (N / 2) + n / 2] = lsb_from_float<T>(moe_gate_mul(acc[j], up, act, limit));
+        } else if (MODE == 2) {
+            if (n < N) ((T*)out_)[(size_t)m * N + n] = lsb_from_float<T>(moe_plain(acc[j], act));
         } else if (n < N) {
             ((float*)out_)[(size_t)m * N + n] = acc[j];
         }
@@ -242,10 +263,12 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict
 template <typename T, typename TY>
 __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restrict__ pos,
                                    const float* __restrict__ wts, int on_output, int top, int n,
-                                   int capacity, T* __restrict__ out, const T* __restrict__ add) {
+                                   int capacity, T* __restrict__ out, const T* __restrict__ add,
+                                   const float* __restrict__ add_gate, int gate_ld) {
     lsb_pdl_launch_dependents();
     lsb_pdl_wait();
     const size_t t = blockIdx.x;
+    const float ag = add_gate ? 1.f / (1.f + expf(-add_gate[t * gate_ld])) : 1.f;
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
         float s = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -254,18 +277,18 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
             const float v = lsb_to_float(y[(size_t)p * n + i]);
             s += on_output ? wts[t * top + k] * v : v;
         }
-        if (add) s += lsb_to_float(add[t * n + i]);          // (what every token passes besides its chosen experts)
+        if (add) s += ag * lsb_to_float(add[t * n + i]);          // (what every token passes besides its chosen experts)
         out[t * n + i] = lsb_from_float<T>(s);
     }
 }
 
 LSB_API int lsb_moe_tile() { return kTile; }
 
-LSB_API int lsb_moe_route(const float* logits, int n_tokens, int E, int top, int score, int renorm,
-                          const float* bias, float scale, float eps, int* ids, float* wts, cudaStream_t stream) {
-    const RouteOpts ro = {score, renorm, bias, scale, eps};
+LSB_API int lsb_moe_route(const float* logits, int ld, int n_tokens, int E, int top, int score, int renorm,
+                          const float* bias, int joins, float scale, float eps, int* ids, float* wts, cudaStream_t stream) {
+    const RouteOpts ro = {score, renorm, bias, scale, eps, joins, ld};
     if (n_tokens <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || top > kMaxTop || score < 0 || score > 1) return (int)cudaErrorInvalidValue;
+    if (E <= 0 || top <= 0 || top > E || top > kMaxTop || score < 0 || score > 2 || ld < E) return (int)cudaErrorInvalidValue;
     const int warps_per_block = 4;
     return lsb_launch(moe_route_kernel, dim3((n_tokens + warps_per_block - 1) / warps_per_block),
                       dim3(32 * warps_per_block), 0, stream, 1, logits, n_tokens, E, top, ro, ids, wts);
@@ -274,13 +297,13 @@ LSB_API int lsb_moe_route(const float* logits, int n_tokens, int E, int top, int
 // logits given (32-bit [tokens, E]): ids and wts are chosen here first (see lsb_moe_route) and written
 LSB_API int lsb_moe_align(int* ids, float* wts, int n_tokens, int top, int E, int cap_tiles,
                           int tile, int* pos, int* row_token, float* row_scale, int* tile_expert,
-                          const float* logits, int score, int renorm, const float* bias, float scale, float eps,
+                          const float* logits, int ld, int score, int renorm, const float* bias, int joins, float scale, float eps,
                           cudaStream_t stream) {
-    const RouteOpts ro = {score, renorm, bias, scale, eps};
+    const RouteOpts ro = {score, renorm, bias, scale, eps, joins, ld};
     if (n_tokens <= 0) return 0;
     const long long n = (long long)n_tokens * top;
     if (E <= 0 || E > 8192 || tile <= 0 || cap_tiles < (n + tile - 1) / tile + E) return (int)cudaErrorInvalidValue;
-    if (logits && (top > kMaxTop || top > E || score < 0 || score > 1)) return (int)cudaErrorInvalidValue;
+    if (logits && (top > kMaxTop || top > E || score < 0 || score > 2 || ld < E)) return (int)cudaErrorInvalidValue;
     return lsb_launch(moe_align_kernel, dim3(1), dim3(1024), (size_t)(2 * E + 1) * sizeof(int), stream, 1,
                       ids, wts, (int)n, top, E, cap_tiles, tile, pos, row_token, row_scale, tile_expert, logits, ro);
 }
@@ -296,12 +319,17 @@ LSB_API int lsb_moe_gather(const void* x, int dtype, const int* pos, const float
     return 0;
 }
 
+// `plain`: w is [E, F, K] and act a plain activation; else [E, 2F, K], gate and up rows alternating
 LSB_API int lsb_moe_up(const void* x, int dtype, const int* row_token, const float* row_scale, int on_input,
                        const void* w, const int* tile_expert, int cap_tiles, void* out, int F, int K,
-                       int act, float limit, cudaStream_t stream) {
+                       int act, float limit, int plain, cudaStream_t stream) {
     if (cap_tiles <= 0) return 0;
     if (F <= 0 || K <= 0 || cap_tiles > 65535) return (int)cudaErrorInvalidValue;
-    dim3 grid((2 * F + kTile - 1) / kTile, cap_tiles);
+    dim3 grid(((plain ? F : 2 * F) + kTile - 1) / kTile, cap_tiles);
+    if (plain)
+        LSB_DISPATCH_DTYPE(dtype, return lsb_launch(moe_gemm_kernel<T, 2>, grid, dim3(256), 0, stream, 1,
+                                                    (const T*)x, row_token, row_scale, on_input, (const T*)w,
+                                                    tile_expert, out, F, K, act, limit));
     LSB_DISPATCH_DTYPE(dtype, return lsb_launch(moe_gemm_kernel<T, 0>, grid, dim3(256), 0, stream, 1,
                                                 (const T*)x, row_token, row_scale, on_input, (const T*)w,
                                                 tile_expert, out, 2 * F, K, act, limit));
@@ -323,14 +351,14 @@ LSB_API int lsb_moe_down(const void* h, int dtype, const int* row_token, const v
 // y_same: the expert rows are stored in the output's type (the tensor-core path), else 32-bit
 LSB_API int lsb_moe_combine(const void* y, int y_same, const int* pos, const float* wts, int on_output,
                             int n_tokens, int top, int n, int capacity, void* out, int dtype, const void* add,
-                            cudaStream_t stream) {
+                            const float* add_gate, int gate_ld, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     LSB_DISPATCH_DTYPE(dtype, {
         if (y_same)
             return lsb_launch(moe_combine_kernel<T, T>, dim3(n_tokens), dim3(256), 0, stream, 1, (const T*)y, pos,
-                              wts, on_output, top, n, capacity, (T*)out, (const T*)add);
+                              wts, on_output, top, n, capacity, (T*)out, (const T*)add, add_gate, gate_ld);
         return lsb_launch(moe_combine_kernel<T, float>, dim3(n_tokens), dim3(256), 0, stream, 1, (const float*)y,
-                          pos, wts, on_output, top, n, capacity, (T*)out, (const T*)add);
+                          pos, wts, on_output, top, n, capacity, (T*)out, (const T*)add, add_gate, gate_ld);
     });
     return 0;
 }

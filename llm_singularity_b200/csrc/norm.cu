@@ -3,6 +3,8 @@
 //   residual[t,:] += delta[t,:]                    (32-bit, in place; delta optional)
 //   out[t,:] = residual[t,:] * rsqrt(mean(residual[t,:]^2) + eps) * weight
 //
+// A second delta of the same shape may join the sum (sublayers that read one input side by side).
+//
 // Replaces residual_add_kernel + rms_norm_kernel of the reference
 // (kernels/src/residual.cu:11-19, kernels/src/rmsnorm.cu:42-72).  The gathered form
 // does the same for selected rows only (the rows whose logits are wanted) and
@@ -17,7 +19,7 @@ constexpr int kNormRegs = 8;          // rows up to 256*8 = 2048 wide stay in re
 
 template <typename T, bool GATHER>
 __global__ void __launch_bounds__(kNormThreads)
-add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
+add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta, const T* __restrict__ delta2,
                    const int* __restrict__ rows, const float* __restrict__ weight,
                    T* __restrict__ out, int hidden, int n_rows_total, float eps) {
     __shared__ float scratch[33];
@@ -36,6 +38,7 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
     }
     float* res = residual + (size_t)r_in * hidden;
     const T* dl = delta ? delta + (size_t)r_in * hidden : nullptr;
+    const T* d2 = delta && delta2 ? delta2 + (size_t)r_in * hidden : nullptr;
     T* o = out + (size_t)r_out * hidden;
 
     float keep[kNormRegs];
@@ -48,7 +51,7 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
             float x = 0.f;
             if (i < hidden) {
                 x = res[i];
-                if (dl) x += lsb_to_float(dl[i]);
+                if (dl) x += d2 ? lsb_to_float(dl[i]) + lsb_to_float(d2[i]) : lsb_to_float(dl[i]);
                 if (!GATHER && dl) res[i] = x;
             }
             keep[j] = x;
@@ -57,7 +60,7 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
     } else {
         for (int i = threadIdx.x; i < hidden; i += kNormThreads) {
             float x = res[i];
-            if (dl) x += lsb_to_float(dl[i]);
+            if (dl) x += d2 ? lsb_to_float(dl[i]) + lsb_to_float(d2[i]) : lsb_to_float(dl[i]);
             if (!GATHER && dl) res[i] = x;
             ss += x * x;
         }
@@ -73,7 +76,7 @@ add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ delta,
     } else {
         for (int i = threadIdx.x; i < hidden; i += kNormThreads) {
             float x = res[i];
-            if (GATHER && dl) x += lsb_to_float(dl[i]);
+            if (GATHER && dl) x += d2 ? lsb_to_float(dl[i]) + lsb_to_float(d2[i]) : lsb_to_float(dl[i]);
             o[i] = lsb_from_float<T>(x * inv * weight[i]);
         }
     }
@@ -104,9 +107,19 @@ template <> struct Vec4<__nv_bfloat16> {
     }
 };
 
+template <typename T>
+__device__ __forceinline__ float4 both(const T* d1, const T* d2, int i) {
+    float4 d = Vec4<T>::load(d1 + i);
+    if (d2) {
+        const float4 e = Vec4<T>::load(d2 + i);
+        d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
+    }
+    return d;
+}
+
 template <typename T, bool GATHER>
 __global__ void __launch_bounds__(kNormThreads)
-add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delta,
+add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delta, const T* __restrict__ delta2,
                         const int* __restrict__ rows, const float* __restrict__ weight,
                         T* __restrict__ out, int hidden, int n_rows_total, float eps) {
     __shared__ float scratch[33];
@@ -137,6 +150,7 @@ add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delt
     }
     float* res = residual + (size_t)r_in * hidden;
     const T* dl = delta ? delta + (size_t)r_in * hidden : nullptr;
+    const T* d2 = delta && delta2 ? delta2 + (size_t)r_in * hidden : nullptr;
     T* o = out + (size_t)r_out * hidden;
     float4 keep[kVecRegs];
     float ss = 0.f;
@@ -148,7 +162,7 @@ add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delt
             if (v < nvec) {
                 x = Vec4<float>::load(res + 4 * v);
                 if (dl) {
-                    const float4 d = Vec4<T>::load(dl + 4 * v);
+                    const float4 d = both<T>(dl, d2, 4 * v);
                     x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
                     if (!GATHER) Vec4<float>::store(res + 4 * v, x);
                 }
@@ -160,7 +174,7 @@ add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delt
         for (int v = threadIdx.x; v < nvec; v += kNormThreads) {
             float4 x = Vec4<float>::load(res + 4 * v);
             if (dl) {
-                const float4 d = Vec4<T>::load(dl + 4 * v);
+                const float4 d = both<T>(dl, d2, 4 * v);
                 x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
                 if (!GATHER) Vec4<float>::store(res + 4 * v, x);
             }
@@ -183,7 +197,7 @@ add_rmsnorm_vec4_kernel(float* __restrict__ residual, const T* __restrict__ delt
         for (int v = threadIdx.x; v < nvec; v += kNormThreads) {
             float4 x = Vec4<float>::load(res + 4 * v);
             if (GATHER && dl) {
-                const float4 d = Vec4<T>::load(dl + 4 * v);
+                const float4 d = both<T>(dl, d2, 4 * v);
                 x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
             }
             const float4 w = Vec4<float>::load(weight + 4 * v);
@@ -198,32 +212,32 @@ static inline bool vec4_ok(const void* a, const void* b, const void* c, const vo
 }
 
 // residual: float [rows, hidden] (updated in place when delta is given)
-// delta: dtype [rows, hidden] or null; weight: float [hidden]; out: dtype [rows, hidden]
-LSB_API int lsb_add_rmsnorm(float* residual, const void* delta, const float* weight, void* out,
+// delta: dtype [rows, hidden] or null; delta2: another one, or null; weight: float [hidden]; out: dtype [rows, hidden]
+LSB_API int lsb_add_rmsnorm(float* residual, const void* delta, const void* delta2, const float* weight, void* out,
                             int dtype, int rows, int hidden, float eps, cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (vec4_ok(residual, delta, weight, out, hidden))
+    if (vec4_ok(residual, delta, weight, out, hidden) && (uintptr_t)delta2 % 16 == 0)
         LSB_DISPATCH_DTYPE(dtype, return lsb_launch(
             add_rmsnorm_vec4_kernel<T, false>, dim3(rows), dim3(kNormThreads), 0, stream, 1,
-            residual, (const T*)delta, (const int*)nullptr, weight, (T*)out, hidden, rows, eps));
+            residual, (const T*)delta, (const T*)delta2, (const int*)nullptr, weight, (T*)out, hidden, rows, eps));
     LSB_DISPATCH_DTYPE(dtype, return lsb_launch(
         add_rmsnorm_kernel<T, false>, dim3(rows), dim3(kNormThreads), 0, stream, 1,
-        residual, (const T*)delta, (const int*)nullptr, weight, (T*)out, hidden, rows, eps));
+        residual, (const T*)delta, (const T*)delta2, (const int*)nullptr, weight, (T*)out, hidden, rows, eps));
     return 0;
 }
 
 // out[i,:] = norm(residual[rows[i],:] + delta[rows[i],:]); residual is not modified.
-LSB_API int lsb_gather_add_rmsnorm(const float* residual, const void* delta, const int* rows,
+LSB_API int lsb_gather_add_rmsnorm(const float* residual, const void* delta, const void* delta2, const int* rows,
                                    const float* weight, void* out, int dtype, int n_out,
                                    int n_rows_total, int hidden, float eps, cudaStream_t stream) {
     if (n_out <= 0) return 0;
-    if (vec4_ok(residual, delta, weight, out, hidden))
+    if (vec4_ok(residual, delta, weight, out, hidden) && (uintptr_t)delta2 % 16 == 0)
         LSB_DISPATCH_DTYPE(dtype, return lsb_launch(
             add_rmsnorm_vec4_kernel<T, true>, dim3(n_out), dim3(kNormThreads), 0, stream, 1,
-            (float*)residual, (const T*)delta, rows, weight, (T*)out, hidden, n_rows_total, eps));
+            (float*)residual, (const T*)delta, (const T*)delta2, rows, weight, (T*)out, hidden, n_rows_total, eps));
     LSB_DISPATCH_DTYPE(dtype, return lsb_launch(
         add_rmsnorm_kernel<T, true>, dim3(n_out), dim3(kNormThreads), 0, stream, 1,
-        (float*)residual, (const T*)delta, rows, weight, (T*)out, hidden, n_rows_total, eps));
+        (float*)residual, (const T*)delta, (const T*)delta2, rows, weight, (T*)out, hidden, n_rows_total, eps));
     return 0;
 }
 

@@ -263,9 +263,18 @@ def embedding_pair(table: torch.Tensor, pair_table: torch.Tensor, ctx, last_toke
           _f(scale), _stream(out))
 
 
+def _check_second_delta(what: str, delta, delta2) -> None:
+    if delta2 is not None:
+        if delta is None:
+            raise KernelError(f"{what}: a second delta without a first")
+        _req(delta2, "delta2", delta.dtype, 2)
+        if delta2.shape != delta.shape:
+            raise KernelError(f"{what}: the deltas have different shapes")
+
+
 def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor,
-                eps: float, out: torch.Tensor) -> None:
-    """residual += delta (in place, 32-bit); out = rmsnorm(residual) * weight."""
+                eps: float, out: torch.Tensor, delta2: Optional[torch.Tensor] = None) -> None:
+    """residual += delta (+ delta2) (in place, 32-bit); out = rmsnorm(residual) * weight."""
     _req(residual, "residual", torch.float32, 2)
     _req(weight, "weight", torch.float32, 1)
     _req(out, "out", dim=2)
@@ -276,13 +285,14 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: t
         _req(delta, "delta", out.dtype, 2)
         if delta.shape != (T, H):
             raise KernelError("add_rmsnorm: delta has another shape than residual")
-    _call("norm", "lsb_add_rmsnorm", _p(residual), _p(delta), _p(weight), _p(out), _i(_dt(out)),
+    _check_second_delta("add_rmsnorm", delta, delta2)
+    _call("norm", "lsb_add_rmsnorm", _p(residual), _p(delta), _p(delta2), _p(weight), _p(out), _i(_dt(out)),
           _i(T), _i(H), _f(eps), _stream(out))
 
 
 def gather_add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], rows: torch.Tensor,
-                       weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
-    """out[i] = rmsnorm(residual[rows[i]] + delta[rows[i]]) * weight; residual unchanged."""
+                       weight: torch.Tensor, eps: float, out: torch.Tensor, delta2: Optional[torch.Tensor] = None) -> None:
+    """out[i] = rmsnorm(residual[rows[i]] + delta[rows[i]] (+ delta2[rows[i]])) * weight; residual unchanged."""
     _req(residual, "residual", torch.float32, 2)
     _req(rows, "rows", torch.int32, 1)
     _req(weight, "weight", torch.float32, 1)
@@ -294,7 +304,8 @@ def gather_add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], ro
         _req(delta, "delta", out.dtype, 2)
         if delta.shape != (T, H):
             raise KernelError("gather_add_rmsnorm: delta has another shape than residual")
-    _call("norm", "lsb_gather_add_rmsnorm", _p(residual), _p(delta), _p(rows), _p(weight), _p(out),
+    _check_second_delta("gather_add_rmsnorm", delta, delta2)
+    _call("norm", "lsb_gather_add_rmsnorm", _p(residual), _p(delta), _p(delta2), _p(rows), _p(weight), _p(out),
           _i(_dt(out)), _i(rows.shape[0]), _i(T), _i(H), _f(eps), _stream(out))
 
 
@@ -304,6 +315,10 @@ ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "none": 3, "capped_glu": 5}     # act(
 # a few rows); where another kernel makes the product (32-bit, sizes those two refuse) it leaves gate and up
 # side by side and the activation kernel follows.
 UNFUSED_GATED = ("capped_glu",)
+# Activations of ungated products that the tensor-core products know in their epilogues (``linear(plain_act=)``):
+# the ids that csrc/activation.cu uses, handed over with _PLAIN added.
+PRODUCT_PLAIN_ACTS = {"silu": 1, "gelu_tanh": 2, "relu_squared": 6}
+_PLAIN = 16
 
 
 def _activation_id(name: str) -> int:
@@ -398,7 +413,7 @@ def finish_norm(x: NormOut) -> torch.Tensor:
 
 
 def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-           gated: bool = False, activation: str = "silu", into=None, limit: float = 0.0):
+           gated: bool = False, activation: str = "silu", into=None, limit: float = 0.0, plain_act: Optional[str] = None):
     """x [M, K] times w [N, K] transposed -> [M, N]; 32-bit accumulation.
 
     ``x`` may be a ``NormOut`` (the norm before this product, possibly half done: see there).
@@ -413,7 +428,12 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
     ``out[m, i] = act(d[m, 2i]) * d[m, 2i + 1]`` (applied in the product's epilogue on the
     tensor-core path, by the activation kernel otherwise); ``activation`` names act: "silu",
     "gelu_tanh", "none", or "capped_glu" with its ``limit``.
+
+    ``plain_act``: an activation on every element of an ungated product ("silu", "gelu_tanh", "relu_squared"),
+    in 32-bit before the result is rounded where a tensor-core kernel makes the product.
     """
+    if plain_act is not None and (gated or into is not None or plain_act not in PRODUCT_PLAIN_ACTS):
+        raise KernelError(f"linear: '{plain_act}' is not an activation of an ungated product")
     if gated and activation in UNFUSED_GATED:
         if into is not None:
             raise KernelError("linear: a product into the residual is plain and in the compute dtype")
@@ -446,6 +466,8 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
         gated_activation(raw, half, activation, limit)
         return half
     act = _activation_id(activation) if gated else 0
+    if plain_act is not None:
+        act = _PLAIN + PRODUCT_PLAIN_ACTS[plain_act]
     owed = None
     if isinstance(x, NormOut):
         owed, x = (x if x.parts is not None else None), x.values
@@ -490,7 +512,7 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
         out = torch.empty_like(delta)
         add_rmsnorm(into[0], delta, into[1], into[2], out)
         return NormOut(out)
-    if x.dtype == torch.bfloat16 and SMALL_PRODUCTS and not gated and M <= 16 and small_gemm_ok(x, w):
+    if x.dtype == torch.bfloat16 and SMALL_PRODUCTS and not act and M <= 16 and small_gemm_ok(x, w):
         # a few rows times a matrix that fits the chip's shared memory (decode: q/k/v, output
         # projection): weights resident before the previous kernel has ended, no cluster
         _chain_ends()
@@ -519,6 +541,8 @@ def linear(x, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
         half = torch.empty((M, N // 2), dtype=out_dtype, device=x.device)
         gated_activation(out, half, activation)
         return half
+    if plain_act is not None:
+        plain_activation(out, out, plain_act)
     return out
 
 
@@ -1316,7 +1340,8 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
                    k_norm=None, norm_eps: float = 0.0, temp_coef: float = 0.0, temp_every: int = 0,
                    inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, pairing: str = "half",
                    store: bool = True, norm_all: bool = False, v_unit: bool = False,
-                   v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None) -> None:
+                   v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
+                   maps: int = 1) -> None:
     """From the rows of ``proj`` (q at ``q_off``, k at ``k_off``, v at ``v_off``) to queries in ``q_out``
     [T, nh * dk] and keys and values in this step's cache places: biases, a norm per head of q and k
     (one weight of head size each), the query temperature ``1 + coef * ln(floor((pos + 1) / every) + 1)``
@@ -1325,17 +1350,21 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
     value head is divided by its root mean square (eps ``norm_eps``, no weight) on its way into the cache.
     ``v_first`` [T, nkv * dv] (rows may be strided) with ``v_lambda`` (one 32-bit number on the device): the
     values are mixed with those another layer made of the same tokens, v <- (1 - lambda) v + lambda v_first,
-    and cached so."""
+    and cached so.  ``maps``: every query and key head is that many parts of ``dk`` side by side, each normed
+    and rotated as a head of its own; q_out is then [T, nh * maps * dk] and a cached key maps * dk long."""
     _req(proj, "proj", dim=2)
     _req(q_out, "q_out", proj.dtype, 2)
     T, ld = proj.shape
-    if ctx.n_tokens != T or q_out.shape != (T, nh * dk):
+    if maps < 1 or (maps > 1 and norm_all):
+        raise KernelError("attention_prep: heads of several maps have no norm over all of them")
+    if ctx.n_tokens != T or q_out.shape != (T, nh * maps * dk):
         raise KernelError("attention_prep: proj, q_out and the step disagree")
-    if min(q_off, k_off, v_off) < 0 or q_off + nh * dk > ld or k_off + nkv * dk > ld or v_off + nkv * dv > ld:
+    if min(q_off, k_off, v_off) < 0 or q_off + nh * maps * dk > ld or k_off + nkv * maps * dk > ld \
+            or v_off + nkv * dv > ld:
         raise KernelError("attention_prep: a projection lies outside the rows of proj")
     if dk > _lib("attention_prep").lsb_attention_prep_max_dim():
         raise KernelError(f"attention_prep: key size {dk} is not supported")
-    for name, t, n in (("q_bias", q_bias, nh * dk), ("k_bias", k_bias, nkv * dk), ("v_bias", v_bias, nkv * dv),
+    for name, t, n in (("q_bias", q_bias, nh * maps * dk), ("k_bias", k_bias, nkv * maps * dk), ("v_bias", v_bias, nkv * dv),
                        ("q_norm", q_norm, nh * dk if norm_all else dk),
                        ("k_norm", k_norm, nkv * dk if norm_all else dk)):
         if t is not None:
@@ -1356,10 +1385,10 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
         if v_first.shape != (T, nkv * dv) or v_first.stride(1) != 1 or v_lambda.numel() != 1 or v_unit:
             raise KernelError("attention_prep: v_first must be [T, kv heads * value size] with one mixing number")
         v_first_ld = v_first.stride(0)
-    _check_kv_cache(cache, nkv, dk, dv, proj.dtype)
+    _check_kv_cache(cache, nkv, maps * dk, dv, proj.dtype)
     _call("attention_prep", "lsb_attention_prep", _p(proj), _i(_dt(proj)), _ll(ld), _i(q_off), _i(k_off), _i(v_off),
           _i(T), _i(nh), _i(nkv), _i(dk), _i(dv), _p(q_bias), _p(k_bias), _p(v_bias), _p(q_norm), _p(k_norm),
-          _f(norm_eps), _i(1 if norm_all else 0), _i(1 if v_unit else 0), _f(temp_coef), _i(temp_every), _p(inv_freq if rotary_dim else None), _i(rotary_dim),
+          _f(norm_eps), _i(1 if norm_all else 0), _i(1 if v_unit else 0), _i(maps), _f(temp_coef), _i(temp_every), _p(inv_freq if rotary_dim else None), _i(rotary_dim),
           _i(_PAIRINGS[pairing]), _p(ctx.positions), _p(ctx.token_req), _p(ctx.table_rows), _p(cache.block_table),
           _i(cache.block_table.shape[1]), _p(q_out), _p(cache.k_pages), _p(cache.v_pages), _i(cache.page_size),
           _i(cache.k_pages.shape[0]), _i(1 if store else 0), _p(v_first), _ll(v_first_ld), _p(v_lambda), _stream(proj))
@@ -1453,6 +1482,58 @@ def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cach
           _stream(out))
 
 
+def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cache, scale: float, window: int,
+                   chunk: int, mixing: torch.Tensor, eps: float, post: float, out: torch.Tensor) -> None:
+    """Differential attention of this step's queries ``q`` [T, nh * 2 * dk] (a head is [map 0 | map 1]) over cached
+    keys [map 0 | map 1] of 2 * dk and values of dv: o = a_0 - ``mixing`` * a_1 with a_m the softmax attention
+    of map m over the head's values (``mixing`` one 32-bit number on the device), and ``out`` [T, nh * dv] is
+    o / sqrt(mean(o^2) + eps) * ``post`` per head.  What a row sees (causal, ``window``, ``chunk``) is as in
+    ``attention_dv``.
+
+    bfloat16 with both sizes multiples of 8 (dk up to 128, dv up to 256) runs on the tensor cores; everything
+    else runs the generic kernel.  Single tokens that stand before a step's portions (as the scheduler puts
+    them) get a launch of their own, shaped for rows that wait on memory."""
+    _req(q, "q", dim=2)
+    _req(out, "out", q.dtype, 2)
+    _req(mixing, "mixing", torch.float32)
+    T = q.shape[0]
+    if q.shape[1] != nh * 2 * dk or out.shape != (T, nh * dv) or ctx.n_tokens != T or mixing.numel() != 1:
+        raise KernelError("attention_diff: q, out, the mixing number and the step disagree")
+    if nkv <= 0 or nh % nkv:
+        raise KernelError(f"attention_diff: {nh} heads cannot share {nkv} kv heads")
+    lib = _lib("attention_diff")
+    if max(2 * dk, dv) > lib.lsb_attention_diff_max_dim():
+        raise KernelError(f"attention_diff: head sizes {dk}, {dv} are not supported")
+    _check_kv_cache(cache, nkv, 2 * dk, dv, q.dtype)
+    common = (_p(cache.block_table), _i(cache.block_table.shape[1]), _p(out))
+    sizes = (_i(nh), _i(nkv), _i(dk), _i(dv), _i(cache.page_size), _i(cache.k_pages.shape[0]), _f(scale), _i(window),
+             _i(chunk), _p(mixing), _f(eps), _f(post))
+    if not (DV_TENSOR_CORES and q.dtype == torch.bfloat16 and lib.lsb_attention_diff_mma_supported(_i(dk), _i(dv))):
+        _call("attention_diff", "lsb_attention_diff_generic", _p(q), _p(cache.k_pages), _p(cache.v_pages), _p(ctx.q_start),
+              _p(ctx.kv_len), _p(ctx.table_rows), *common, _i(_dt(q)), _i(ctx.n_requests), _i(ctx.max_q_len), *sizes,
+              _stream(out))
+        return
+    spans = [(0, ctx.n_requests, ctx.max_q_len)]
+    if ctx.max_q_len > 1:
+        n_decode, first, last = _batch_shape(ctx)
+        if n_decode and n_decode == first and last == ctx.n_requests:
+            spans = [(0, first, 1), (first, ctx.n_requests - first, ctx.max_q_len)]
+    sms = num_sms(q.device)
+    for at, n_req, max_q in spans:
+        plan = lib.lsb_attention_diff_plan(_i(n_req), _i(max_q), _i(nh), _i(nkv), _i(chunk), _i(sms), _i(DV_BLOCK_SHAPE))
+        scratch = None
+        if plan >> 8 > 1:
+            tiles = -(-max_q * (nh // nkv) // 16)
+            key = ("attention_diff", q.device, n_req * nkv * tiles * (plan >> 8) * 16 * 2 * (dv + 2))
+            scratch = _scratch.get(key)
+            if scratch is None:
+                scratch = _scratch[key] = torch.empty(key[2], dtype=torch.float32, device=q.device)
+        _call("attention_diff", "lsb_attention_diff_mma", _p(q), _p(cache.k_pages), _p(cache.v_pages),
+              ctypes.c_void_p(ctx.q_start.data_ptr() + 4 * at), ctypes.c_void_p(ctx.kv_len.data_ptr() + 4 * at),
+              ctypes.c_void_p(ctx.table_rows.data_ptr() + 4 * at), *common, _i(n_req), _i(max_q), *sizes, _i(sms),
+              _i(DV_BLOCK_SHAPE), _p(scratch), _stream(out))
+
+
 def branch_sum(ys, scales, out: torch.Tensor) -> None:
     """out = sum_b scales[b] * ys[b], summed in 32-bit (mixers side by side whose results are added
     with fixed factors)."""
@@ -1470,12 +1551,12 @@ def branch_sum(ys, scales, out: torch.Tensor) -> None:
           _stream(out))
 
 
-PLAIN_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "none": 3, "bent_square": 4}
+PLAIN_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2, "none": 3, "bent_square": 4, "relu_squared": 6}
 
 
 def plain_activation(x: torch.Tensor, out: torch.Tensor, activation: str, c_pos: float = 0.0, c_neg: float = 0.0) -> None:
     """out = act(x) element by element, evaluated in 32-bit.  "bent_square": ``c_pos z^2 + z/2`` right of
-    zero, ``c_neg (e^z - 1 - z) + z/2`` left of it."""
+    zero, ``c_neg (e^z - 1 - z) + z/2`` left of it.  "relu_squared": ``max(z, 0)^2``.  ``out`` may be ``x``."""
     _req(x, "x")
     _req(out, "out", x.dtype)
     if out.shape != x.shape or activation not in PLAIN_ACTIVATIONS:
@@ -1701,7 +1782,7 @@ def memory_output(walked: torch.Tensor, floor: torch.Tensor, weight: torch.Tenso
 
 
 # ------------------------------------------------------------------------ routed experts
-MOE_SCORES = {"sigmoid": 0, "softmax": 1}
+MOE_SCORES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
 MOE_TENSOR_CORES = True         # bfloat16 experts on the grouped tcgen05 product
 
 
@@ -1710,28 +1791,30 @@ def moe_tile() -> int:
     return int(_lib("moe").lsb_moe_tile())
 
 
-def _route_options(E: int, choice_bias: Optional[torch.Tensor], weight_scale: float, renorm_eps: float):
+def _route_options(E: int, choice_bias: Optional[torch.Tensor], weight_scale: float, renorm_eps: float, joins: bool = False):
     if choice_bias is not None:
         _req(choice_bias, "choice_bias", torch.float32, 1)
         if choice_bias.shape[0] != E:
-            raise KernelError(f"moe: the choice bias must have {E} entries")
-    return _p(choice_bias), _f(weight_scale), _f(renorm_eps)
+            raise KernelError(f"moe: the router's bias must have {E} entries")
+    return _p(choice_bias), _i(1 if joins else 0), _f(weight_scale), _f(renorm_eps)
 
 
 def moe_route(logits: torch.Tensor, top: int, score: str, renormalize: bool, ids: torch.Tensor,
               weights: torch.Tensor, choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
-              renorm_eps: float = 0.0) -> None:
+              renorm_eps: float = 0.0, bias_in_logits: bool = False) -> None:
     """The ``top`` experts with the largest scores per row of 32-bit ``logits`` and their scores.
     ``choice_bias`` (one number an expert) is added to the scores for the choice only; the weights are the
-    chosen scores themselves, divided by their sum + ``renorm_eps`` if ``renormalize``, times ``weight_scale``."""
+    chosen scores themselves, divided by their sum + ``renorm_eps`` if ``renormalize``, times ``weight_scale``.
+    ``score`` "softmax_chosen": the weights are the softmax over the chosen logits alone.  ``bias_in_logits``: the
+    bias is part of the logits, for the choice and for the weights."""
     _req(logits, "logits", torch.float32, 2)
     _req(ids, "ids", torch.int32, 2)
     _req(weights, "weights", torch.float32, 2)
     T, E = logits.shape
     if ids.shape != (T, top) or weights.shape != (T, top) or not 0 < top <= min(E, 32):
         raise KernelError("moe_route: ids / weights must be [tokens, top], top at most 32")
-    _call("moe", "lsb_moe_route", _p(logits), _i(T), _i(E), _i(top), _i(MOE_SCORES[score]),
-          _i(1 if renormalize else 0), *_route_options(E, choice_bias, weight_scale, renorm_eps), _p(ids), _p(weights),
+    _call("moe", "lsb_moe_route", _p(logits), _i(E), _i(T), _i(E), _i(top), _i(MOE_SCORES[score]),
+          _i(1 if renormalize else 0), *_route_options(E, choice_bias, weight_scale, renorm_eps, bias_in_logits), _p(ids), _p(weights),
           _stream(ids))
 
 
@@ -1741,32 +1824,39 @@ MOE_FUSED_ROUTING_TOKENS = 256  # steps of at most this many tokens choose their
 def moe_routed_experts(x: torch.Tensor, logits: torch.Tensor, top: int, score: str, renormalize: bool,
                        w_gate_up: torch.Tensor, w_down: torch.Tensor, activation: str, weight_on: str,
                        out: torch.Tensor, choice_bias: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
-                       renorm_eps: float = 0.0, limit: float = 0.0, add: Optional[torch.Tensor] = None) -> None:
+                       renorm_eps: float = 0.0, limit: float = 0.0, add: Optional[torch.Tensor] = None,
+                       gated: bool = True, bias_in_logits: bool = False, gate_column: bool = False) -> None:
     """``moe_route`` on the 32-bit ``logits`` followed by ``moe_experts``; in a step of few tokens the
-    choosing rides in the kernel that sorts the rows by expert (one launch less)."""
+    choosing rides in the kernel that sorts the rows by expert (one launch less).  ``gate_column``: the
+    logits have one column more than there are experts, and its sigmoid multiplies ``add``."""
     _req(logits, "logits", torch.float32, 2)
-    T, E = logits.shape
+    T, E = x.shape[0], w_gate_up.shape[0]
+    if logits.shape != (T, E + (1 if gate_column else 0)):
+        raise KernelError("moe_routed_experts: the router's logits must be [tokens, experts] (and the gate's column)")
     ids = torch.empty(T, top, dtype=torch.int32, device=x.device)
     weights = torch.empty(T, top, dtype=torch.float32, device=x.device)
     if not 0 < top <= min(E, 32):
         raise KernelError("moe_routed_experts: top must be in [1, min(experts, 32)]")
-    if T <= MOE_FUSED_ROUTING_TOKENS:
-        moe_experts(x, ids, weights, w_gate_up, w_down, activation, weight_on, out,
-                    route=(logits, MOE_SCORES[score], 1 if renormalize else 0, choice_bias, weight_scale, renorm_eps),
-                    limit=limit, add=add)
-    else:
-        moe_route(logits, top, score, renormalize, ids, weights, choice_bias, weight_scale, renorm_eps)
-        moe_experts(x, ids, weights, w_gate_up, w_down, activation, weight_on, out, limit=limit, add=add)
+    add_gate = logits[:, E:] if gate_column else None
+    route = (logits, MOE_SCORES[score], 1 if renormalize else 0, choice_bias, weight_scale, renorm_eps, bias_in_logits)
+    if T > MOE_FUSED_ROUTING_TOKENS:
+        _call("moe", "lsb_moe_route", _p(logits), _i(logits.shape[1]), _i(T), _i(E), _i(top), _i(route[1]), _i(route[2]),
+              *_route_options(E, choice_bias, weight_scale, renorm_eps, bias_in_logits), _p(ids), _p(weights), _stream(ids))
+        route = None
+    moe_experts(x, ids, weights, w_gate_up, w_down, activation, weight_on, out, route=route, limit=limit, add=add,
+                gated=gated, add_gate=add_gate)
 
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, activation: str, weight_on: str, out: torch.Tensor, route=None,
-                limit: float = 0.0, add: Optional[torch.Tensor] = None) -> None:
+                limit: float = 0.0, add: Optional[torch.Tensor] = None, gated: bool = True,
+                add_gate: Optional[torch.Tensor] = None) -> None:
     """out[t] = sum over k of down_e(act(gate_e u) * up_e u), e = ids[t, k], with u = weights[t, k] * x[t]
     (``weight_on`` "input") or u = x[t] and the sum weighted ("output"); plus ``add[t]`` if given (a shared
     expert's rows, or a callable that makes them: it is called behind the experts' products), in the same
-    32-bit sum.  ``w_gate_up`` [E, 2F, H] has
-    rows alternating gate_i, up_i; ``w_down`` [E, H, F]."""
+    32-bit sum, times sigmoid(``add_gate[t, 0]``) if that is given (32-bit, rows may be strided).
+    ``w_gate_up`` [E, 2F, H] has rows alternating gate_i, up_i; ``w_down`` [E, H, F].  ``gated`` False: the
+    experts are down_e(act(up_e u)) and ``w_gate_up`` is [E, F, H], the up matrices alone."""
     _req(x, "x", dim=2)
     _req(ids, "ids", torch.int32, 2)
     _req(weights, "weights", torch.float32, 2)
@@ -1774,11 +1864,19 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     _req(w_down, "w_down", x.dtype, 3)
     _req(out, "out", x.dtype, 2)
     T, H = x.shape
-    E, F2, _ = w_gate_up.shape
-    F, top = F2 // 2, ids.shape[1]
-    if w_gate_up.shape != (E, 2 * F, H) or w_down.shape != (E, H, F) or out.shape != (T, H) \
+    E, N_up, _ = w_gate_up.shape
+    F, top = N_up // 2 if gated else N_up, ids.shape[1]
+    if w_gate_up.shape != (E, 2 * F if gated else F, H) or w_down.shape != (E, H, F) or out.shape != (T, H) \
             or ids.shape[0] != T or weights.shape != ids.shape or weight_on not in ("input", "output"):
         raise KernelError("moe_experts: shapes disagree")
+    if gated:
+        act = _activation_id(activation)
+        if activation in UNFUSED_GATED and not limit > 0:
+            raise KernelError(f"moe_experts: '{activation}' needs a positive limit")
+    elif activation not in PRODUCT_PLAIN_ACTS:
+        raise KernelError(f"moe_experts: '{activation}' is not an activation of ungated experts")
+    else:
+        act = PRODUCT_PLAIN_ACTS[activation]
     # bfloat16 with TMA-friendly sizes: rows gathered in place, two grouped tcgen05 products over
     # 128-row tiles; anything else (32-bit, odd sizes): the plain grouped kernels over 32-row tiles
     tc = MOE_TENSOR_CORES and x.dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0
@@ -1793,28 +1891,25 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     y = torch.empty(cap_tiles * tile, H, dtype=x.dtype if tc else torch.float32, device=dev)
     s = _stream(out)
     on_input = 1 if weight_on == "input" else 0
-    r_logits, r_score, r_renorm, r_bias, r_scale, r_eps = (tuple(route) + (None, 1.0, 0.0))[:6] if route is not None \
-        else (None, 0, 0, None, 1.0, 0.0)
-    if r_logits is not None and r_logits.shape != (T, E):
+    r_logits, r_score, r_renorm, r_bias, r_scale, r_eps, r_joins = (tuple(route) + (None, 1.0, 0.0, False)[len(route) - 3:])[:7] \
+        if route is not None else (None, 0, 0, None, 1.0, 0.0, False)
+    if r_logits is not None and (r_logits.shape[0] != T or r_logits.shape[1] < E):
         raise KernelError("moe_experts: the router's logits must be [tokens, experts]")
-    unfused = activation in UNFUSED_GATED
-    if unfused and not limit > 0:
-        raise KernelError(f"moe_experts: '{activation}' needs a positive limit")
     _call("moe", "lsb_moe_align", _p(ids), _p(weights), _i(T), _i(top), _i(E), _i(cap_tiles), _i(tile), _p(pos),
-          _p(row_token), _p(row_scale), _p(tile_expert), _p(r_logits), _i(r_score), _i(r_renorm),
-          *_route_options(E, r_bias, r_scale, r_eps), s)
+          _p(row_token), _p(row_scale), _p(tile_expert), _p(r_logits), _i(E if r_logits is None else r_logits.shape[1]),
+          _i(r_score), _i(r_renorm), *_route_options(E, r_bias, r_scale, r_eps, r_joins), s)
     if tc:
         rows = torch.empty(cap_tiles * tile, H, dtype=x.dtype, device=dev)
         _call("moe", "lsb_moe_gather", _p(x), _i(_dt(x)), _p(pos), _p(weights), _i(on_input), _i(T), _i(top),
               _i(cap_tiles * tile), _i(H), _p(rows), s)
         _chain_ends()
         _call("gemm_tc", "lsb_gemm_tc_grouped", _p(rows), _p(w_gate_up), _p(hidden), _i(0), _i(cap_tiles * tile),
-              _i(2 * F), _i(H), _i(E), _p(tile_expert), _i(_activation_id(activation)), _f(limit), s)
+              _i(N_up), _i(H), _i(E), _p(tile_expert), _i(act if gated else _PLAIN + act), _f(limit), s)
         _call("gemm_tc", "lsb_gemm_tc_grouped", _p(hidden), _p(w_down), _p(y), _i(0), _i(cap_tiles * tile),
               _i(H), _i(F), _i(E), _p(tile_expert), _i(0), _f(0.0), s)
     else:
         _call("moe", "lsb_moe_up", _p(x), _i(_dt(x)), _p(row_token), _p(row_scale), _i(on_input), _p(w_gate_up),
-              _p(tile_expert), _i(cap_tiles), _p(hidden), _i(F), _i(H), _i(_activation_id(activation)), _f(limit), s)
+              _p(tile_expert), _i(cap_tiles), _p(hidden), _i(F), _i(H), _i(act), _f(limit), _i(0 if gated else 1), s)
         _call("moe", "lsb_moe_down", _p(hidden), _i(_dt(x)), _p(row_token), _p(w_down), _p(tile_expert), _i(cap_tiles),
               _p(y), _i(H), _i(F), s)
     if callable(add):           # made now, behind the experts' products (its own products' weights are then the
@@ -1823,8 +1918,14 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         _req(add, "add", x.dtype, 2)
         if add.shape != (T, H):
             raise KernelError("moe_experts: add must have out's shape")
+    gate_ld = 0
+    if add_gate is not None:
+        _req(add_gate, "add_gate", torch.float32, 2, contiguous=False)
+        if add is None or add_gate.shape != (T, 1):
+            raise KernelError("moe_experts: the gate is one number a token of rows to add")
+        gate_ld = add_gate.stride(0)
     _call("moe", "lsb_moe_combine", _p(y), _i(1 if tc else 0), _p(pos), _p(weights), _i(1 - on_input), _i(T), _i(top),
-          _i(H), _i(cap_tiles * tile), _p(out), _i(_dt(out)), _p(add), s)
+          _i(H), _i(cap_tiles * tile), _p(out), _i(_dt(out)), _p(add), _p(add_gate), _i(gate_ld), s)
 
 
 def sample(logits: torch.Tensor, params: torch.Tensor, top_k: torch.Tensor,

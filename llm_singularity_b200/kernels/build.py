@@ -48,6 +48,7 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     "sandwich": "sandwich.cu",
     "attention_prep": "attention_prep.cu",
     "attention_dv": "attention_dv.cu",
+    "attention_diff": "attention_diff.cu",
     "matrix_memory": "matrix_memory.cu",
     "delta_rule": "delta_rule.cu",
     "rglru": "rglru.cu",
@@ -56,7 +57,7 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     # host code only: pools, block tables, prefix tree; scheduler
     "host_runtime": ("host_memory.cpp", "host_scheduler.cpp", "host_step.cpp"),
 }
-HEADERS = ["common.cuh", "attention_tc_noalloc.h", "stream_warm.cuh"]     # of the CUDA libraries
+HEADERS = ["common.cuh", "attention_tc_noalloc.h", "attention_dv.cuh", "stream_warm.cuh"]     # of the CUDA libraries
 HOST_HEADERS = ["host_memory.h"]                          # of the host runtime
 
 

@@ -13,7 +13,7 @@ from typing import Dict, Optional
 import torch
 
 from .base import FEED_FORWARDS, MIXERS, NORMS, ParamSpec, Part, register_block
-from .norm import StreamCopy
+from .norm import DeltaPair, StreamCopy
 
 
 @register_block("pre_norm")
@@ -75,6 +75,35 @@ class PreNormBlock(Part):
         if fold and next_norm is not None and self.ffn.folds_norm:
             return self.ffn.forward(self._input(h, self.ffn), ctx, into=(residual, *next_norm.fold()))
         return self.ffn.forward(self._input(h, self.ffn), ctx)
+
+
+@register_block("side_by_side")
+class SideBySideBlock(Part):
+    """``h = norm(x); x += mixer(h) + ffn(h)``: one norm, whose output both sublayers read.  The stream is
+    32-bit and updated in place; neither sublayer's output is added here: both are handed on as a
+    ``DeltaPair``, and the kernel of the norm that comes next (the next block's, or the head's) adds them
+    to the stream in one pass."""
+
+    graph_safe = True
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.norm = NORMS.build(spec.norm, rt)
+        self.mixer = MIXERS.build(spec.mixer, rt)
+        self.ffn = FEED_FORWARDS.build(spec.ffn, rt) if spec.ffn is not None else None
+
+    def children(self) -> Dict[str, Part]:
+        c = {"norm": self.norm, "mixer": self.mixer}
+        if self.ffn is not None:
+            c["ffn"] = self.ffn
+        return c
+
+    def forward(self, residual: torch.Tensor, pending, ctx, cache, writes_cache: bool = True):
+        h = self.norm.add_norm(residual, pending)
+        y = self.mixer.forward(h, ctx, cache, writes_cache)
+        if self.ffn is None:
+            return y
+        return DeltaPair(y, self.ffn.forward(h, ctx))
 
 
 class TokenSide(Part):

@@ -14,7 +14,10 @@ and a gate of one number per head (``gate_per_head``); scores capped by ``cap * 
 (``logit_softcap``) and lowered in proportion to the key's distance with a slope per head
 (``linear_bias``); and values shared within a token among the layers of a model that name the same
 ``value_mix_key``: the "source" layer lends the rows of its value projection to the step
-(``ctx.lent``), a "mixed" layer caches ``(1 - lambda) v + lambda v_source``.
+(``ctx.lent``), a "mixed" layer caches ``(1 - lambda) v + lambda v_source``.  With ``diff`` a head attends twice
+to its values (two queries and keys side by side, one cached row) and the kernels of
+``csrc/attention_diff.cu`` leave the normed difference of the two; the number that multiplies the second
+map is formed once at load, in 64-bit, from the layer's four vectors.
 
 Where the spec is what the framework's grouped attention already covers after the preparation (keys
 and values of one size, no chunks, no gate), the same attention kernels run (tensor cores for
@@ -57,19 +60,26 @@ class KVAttention(Part):
             raise ValueError(f"value_mix '{self.value_mix}' is not known (source, mixed)")
         if self.value_mix and (s.qkv_bias or self.v_unit):
             raise ValueError("values that layers share are neither biased nor normed")
+        self.diff = getattr(s, "diff", None)
+        if self.diff is not None and (s.qkv_bias or s.qk_norm or s.temp_every or s.out_gate or self.v_unit or self.sink
+                                      or self.softcap or self.linear_bias or self.value_mix):
+            raise ValueError("differential attention goes with a position encoding, a window and chunks only")
+        self.maps = 1 if self.diff is None else 2
         self.position = POSITIONS.build(s.position, rt)
         self.table = self.position.rotary_table()
         if self.table is None and s.position.kind != "none":
             raise ValueError(f"a position encoding of kind '{s.position.kind}' is not a rotation this mixer can fuse")
         self.pairing = getattr(s.position, "pairing", "half")
-        self.q_size = s.num_heads * s.key_dim
-        self.k_size = s.num_kv_heads * s.key_dim
+        self.q_size = s.num_heads * s.key_dim * self.maps
+        self.k_size = s.num_kv_heads * s.key_dim * self.maps
         self.v_size = s.num_kv_heads * s.value_dim
         self.o_size = s.num_heads * s.value_dim
         # the framework's grouped attention takes over where nothing here is beyond it
         self.plain = (s.key_dim == s.value_dim and s.chunk is None and not s.out_gate and s.key_dim % 16 == 0
-                      and 16 <= s.key_dim <= 256 and not self.sink and not self.softcap and not self.linear_bias)
-        if self.plain:
+                      and 16 <= s.key_dim <= 256 and self.diff is None and not self.sink and not self.softcap and not self.linear_bias)
+        if self.diff is not None:
+            self.kernels = ("gemm", "attention_prep", "attention_diff")
+        elif self.plain:
             self.kernels = self.kernels + ("attention",)
             if rt.dtype == torch.bfloat16 and s.key_dim in (64, 128):
                 self.kernels = self.kernels + ("attention_tc", "attention_tc5")
@@ -81,7 +91,8 @@ class KVAttention(Part):
     @classmethod
     def params(cls, spec) -> Dict[str, ParamSpec]:
         s, H = spec, spec.hidden_size
-        q, k, v, o = s.num_heads * s.key_dim, s.num_kv_heads * s.key_dim, s.num_kv_heads * s.value_dim, \
+        maps = 1 if getattr(s, "diff", None) is None else 2
+        q, k, v, o = maps * s.num_heads * s.key_dim, maps * s.num_kv_heads * s.key_dim, s.num_kv_heads * s.value_dim, \
             s.num_heads * s.value_dim
         p = {"q": ParamSpec((q, H)), "k": ParamSpec((k, H)), "v": ParamSpec((v, H)), "o": ParamSpec((H, o))}
         if s.qkv_bias:
@@ -96,6 +107,8 @@ class KVAttention(Part):
             p["g"] = ParamSpec((s.num_heads if getattr(s, "gate_per_head", False) else o, H))
         if getattr(s, "value_mix", None) == "mixed":
             p["vmix"] = ParamSpec((), role="vector", init="normal")
+        if maps == 2:
+            p.update({n: ParamSpec((s.key_dim,), role="vector", init="normal") for n in ("lq1", "lk1", "lq2", "lk2")})
         return p
 
     def children(self):
@@ -107,10 +120,16 @@ class KVAttention(Part):
         self.w_out = tensors["o"].contiguous()
         self.extras = {n: tensors[n].contiguous() for n in ("q_bias", "k_bias", "v_bias", "q_norm", "k_norm")
                        if n in tensors}
+        if self.diff is not None:
+            lq1, lk1, lq2, lk2 = (tensors[n].detach().to("cpu", torch.float64) for n in ("lq1", "lk1", "lq2", "lk2"))
+            mixing = torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + float(self.diff)
+            self.mixing = mixing.to(torch.float32).reshape(1).to(self.rt.device)
         self.v_lambda = tensors["vmix"].reshape(1).contiguous() if "vmix" in tensors else None
 
     def cache_spec(self):
         s = self.spec
+        if self.diff is not None:
+            return PagedKVSpec(s.num_kv_heads, 2 * s.key_dim, s.window, s.value_dim)
         return PagedKVSpec(s.num_kv_heads, s.key_dim, s.window, None if s.value_dim == s.key_dim else s.value_dim)
 
     def forward(self, x, ctx, cache, writes_cache: bool = True):
@@ -133,7 +152,10 @@ class KVAttention(Part):
                            temp_every=s.temp_every, inv_freq=inv_freq, rotary_dim=rotary_dim, pairing=self.pairing,
                            store=writes_cache, **self.extras, **self._prep_options(ctx))
         out = self.rt.empty(T, self.o_size)
-        if self.plain:
+        if self.diff is not None:
+            ops.attention_diff(q, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim, ctx, cache, s.scale, s.window or 0,
+                               s.chunk or 0, self.mixing, s.eps, 1.0 - self.diff, out)
+        elif self.plain:
             ops.paged_attention(q, s.num_heads, s.num_kv_heads, s.key_dim, ctx, cache, s.scale, s.window or 0, out)
         else:
             gate = proj[:, self.q_size + self.k_size + self.v_size:] if s.out_gate else None
@@ -150,6 +172,8 @@ class KVAttention(Part):
             opts["norm_all"] = True
         if self.v_unit:
             opts["v_unit"] = True
+        if self.maps > 1:
+            opts["maps"] = self.maps
         return opts
 
     def _softmax_options(self) -> dict:

@@ -52,9 +52,12 @@ class DenseMLP(Part):
 
     def forward(self, x, ctx, into=None):
         ops = self.rt.ops
-        z = ops.linear(x, self.w_up)
-        a = self.rt.empty(*z.shape)
-        ops.plain_activation(z, a, self.spec.activation, self.c_pos, self.c_neg)
+        if self.spec.activation in getattr(ops, "PRODUCT_PLAIN_ACTS", ()):
+            a = ops.linear(x, self.w_up, plain_act=self.spec.activation)        # (in the product's epilogue)
+        else:
+            z = ops.linear(x, self.w_up)
+            a = self.rt.empty(*z.shape)
+            ops.plain_activation(z, a, self.spec.activation, self.c_pos, self.c_neg)
         return ops.linear(a, self.w_down)
 
 

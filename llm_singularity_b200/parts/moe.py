@@ -1,14 +1,17 @@
-"""Routed feed-forward: every token is sent through ``top`` of ``num_experts`` small gated
-feed-forwards, ``down_e(act(gate_e u) * up_e u)``, no bias.
+"""Routed feed-forward: every token is sent through ``top`` of ``num_experts`` small
+feed-forwards, ``down_e(act(gate_e u) * up_e u)`` or, ungated, ``down_e(act(up_e u))``, no bias.
 
 The router is one product with 32-bit output; its logits become scores (sigmoid, or softmax
 over all experts), the ``top`` largest are chosen (the lower index wins a tie) and, if the spec
 says so, divided by their sum.  A score multiplies what the spec names: the expert's input
 (``u = s x``; with a gated expert that is not the same as scaling its output) or its output.
 With ``choice_bias`` a learnt number per expert joins the scores for the choice only; the chosen
-scores are divided by their sum + ``renorm_eps`` and multiplied by ``weight_scale``.  ``shared``: a
-gated feed-forward that every token passes besides its chosen experts; its rows join the 32-bit sum
-over the chosen experts' rows in the combining kernel.
+scores are divided by their sum + ``renorm_eps`` and multiplied by ``weight_scale``.  Score "softmax_chosen"
+is the softmax over the chosen logits alone; ``router_bias`` adds a learnt number per expert to the
+logits, for the choice and the weights.  ``shared``: a feed-forward that every token passes besides its
+chosen experts; its rows join the 32-bit sum over the chosen experts' rows in the combining kernel,
+with ``shared_gate`` multiplied by the sigmoid of one more 32-bit logit per token, whose row of weights
+stands behind the router's in one matrix.
 
 The experts' matrices are stacked (``[E, 2F, H]`` with rows alternating gate_i, up_i, and
 ``[E, H, F]``); a step's (token, choice) pairs are sorted by expert on the device into row
@@ -35,13 +38,19 @@ class RoutedExperts(Part):
         s = spec
         if not 0 < s.top <= s.num_experts:
             raise ValueError(f"top {s.top} of {s.num_experts} experts")
-        if s.score not in ("sigmoid", "softmax") or s.weight_on not in ("input", "output"):
+        if s.score not in ("sigmoid", "softmax", "softmax_chosen") or s.weight_on not in ("input", "output"):
             raise ValueError(f"score '{s.score}' / weight_on '{s.weight_on}' is not known")
-        known = getattr(rt.ops, "ACTIVATIONS", None)
+        self.gated = bool(getattr(s, "gated", True))
+        known = getattr(rt.ops, "ACTIVATIONS" if self.gated else "PRODUCT_PLAIN_ACTS", None)
         if known is not None and s.activation not in known:
             raise ValueError(f"activation '{s.activation}' is not implemented")
         shared = getattr(s, "shared", None)
         self.shared = FEED_FORWARDS.build(shared, rt) if shared is not None else None
+        self.shared_gate = bool(getattr(s, "shared_gate", False))
+        if self.shared_gate and self.shared is None:
+            raise ValueError("a shared expert's gate without a shared expert")
+        if getattr(s, "router_bias", False) and getattr(s, "choice_bias", False):
+            raise ValueError("a router's bias is part of the logits or for the choice alone, not both")
         if self.shared is not None:
             self.kernels = self.kernels + ("activation",)
 
@@ -54,8 +63,13 @@ class RoutedExperts(Part):
         p = {"router": ParamSpec((spec.num_experts, H))}
         if getattr(spec, "choice_bias", False):
             p["choice_bias"] = ParamSpec((spec.num_experts,), role="vector", init="normal")
+        if getattr(spec, "router_bias", False):
+            p["router_bias"] = ParamSpec((spec.num_experts,), role="vector", init="normal")
+        if getattr(spec, "shared_gate", False):
+            p["shared_gate"] = ParamSpec((1, H))
         for e in range(spec.num_experts):
-            p[f"e{e}.gate"] = ParamSpec((F, H))
+            if getattr(spec, "gated", True):
+                p[f"e{e}.gate"] = ParamSpec((F, H))
             p[f"e{e}.up"] = ParamSpec((F, H))
             p[f"e{e}.down"] = ParamSpec((H, F))
         return p
@@ -64,9 +78,12 @@ class RoutedExperts(Part):
         s = self.spec
         E, F, H = s.num_experts, s.expert_size, s.hidden_size
         self.w_router = tensors["router"].contiguous()
+        if self.shared_gate:                        # the gate's row rides behind the router's
+            self.w_router = torch.cat([tensors["router"], tensors["shared_gate"]]).contiguous()
         self.choice_bias = tensors["choice_bias"].contiguous() if "choice_bias" in tensors else None
+        self.router_bias = tensors["router_bias"].contiguous() if "router_bias" in tensors else None
         # rows 2i, 2i + 1 of an expert = gate_i, up_i
-        self.w_gate_up = torch.stack(
+        self.w_gate_up = torch.stack([tensors[f"e{e}.up"] for e in range(E)]).contiguous() if not self.gated else torch.stack(
             [torch.stack([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], dim=1).reshape(2 * F, H) for e in range(E)]
         ).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
@@ -78,6 +95,12 @@ class RoutedExperts(Part):
         extra = {}
         if self.choice_bias is not None:
             extra["choice_bias"] = self.choice_bias
+        if self.router_bias is not None:
+            extra.update(choice_bias=self.router_bias, bias_in_logits=True)
+        if not self.gated:
+            extra["gated"] = False
+        if self.shared_gate:
+            extra["gate_column"] = True
         for name, default in (("weight_scale", 1.0), ("renorm_eps", 0.0), ("limit", 0.0)):
             if getattr(s, name, default) != default:
                 extra[name] = float(getattr(s, name))

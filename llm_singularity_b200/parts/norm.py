@@ -26,6 +26,16 @@ class NormedDelta:
         self.values, self.weight, self.eps, self.mult = values, weight, float(eps), float(mult)
 
 
+class DeltaPair:
+    """Two sublayers' outputs that both still have to join the stream (sublayers that read one input side by
+    side).  Handed on in place of a plain delta: the norm that takes it adds both in 32-bit."""
+
+    __slots__ = ("first", "second")
+
+    def __init__(self, first: torch.Tensor, second: torch.Tensor):
+        self.first, self.second = first, second
+
+
 @register_norm("rmsnorm")
 class RMSNorm(Part):
     """``unit_offset`` in the spec: the checkpoint stores the weight's distance from one; one is added
@@ -74,13 +84,18 @@ class RMSNorm(Part):
         return self.weight, self.spec.eps
 
     def add_norm(self, residual: torch.Tensor, delta, step: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """``delta``: a tensor, None, a ``NormedDelta`` or a ``StreamCopy`` (nothing pending).  ``step``: a
+        """``delta``: a tensor, None, a ``NormedDelta``, a ``DeltaPair`` or a ``StreamCopy`` (nothing pending).  ``step``: a
         vector added to every row of the stream with the sum."""
         if isinstance(delta, StreamCopy):
             delta = None
+        if isinstance(delta, DeltaPair) and step is not None:
+            raise ValueError("a step vector and the outputs of two sublayers cannot join the stream in one sum")
         if isinstance(delta, NormedDelta) or step is not None:
             return self._stream(residual, delta, step, None)
         out = self.rt.empty(*residual.shape)
+        if isinstance(delta, DeltaPair):
+            self.rt.ops.add_rmsnorm(residual, delta.first, self.weight, self.spec.eps, out, delta2=delta.second)
+            return out
         self.rt.ops.add_rmsnorm(residual, delta, self.weight, self.spec.eps, out)
         return out
 
@@ -90,6 +105,9 @@ class RMSNorm(Part):
         if isinstance(delta, NormedDelta):
             return self._stream(residual, delta, None, rows)
         out = self.rt.empty(rows.shape[0], residual.shape[1])
+        if isinstance(delta, DeltaPair):
+            self.rt.ops.gather_add_rmsnorm(residual, delta.first, rows, self.weight, self.spec.eps, out, delta2=delta.second)
+            return out
         self.rt.ops.gather_add_rmsnorm(residual, delta, rows, self.weight, self.spec.eps, out)
         return out
 

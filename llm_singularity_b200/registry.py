@@ -113,6 +113,8 @@ def _register_builtin() -> None:
     register_architecture(FikizenConfig.architecture, FikizenConfig)
     from .config.zinizen import ZinizenConfig
     register_architecture(ZinizenConfig.architecture, ZinizenConfig)
+    from .config.mofidra import MofidraConfig
+    register_architecture(MofidraConfig.architecture, MofidraConfig)
 
 
 _register_builtin()
