@@ -1,4 +1,10 @@
-"""Prefill and decode throughput of a design (Ridotar, Fogezen, Fikizen, Zinizen) beside the Llama decoder at equal size.
+"""Prefill and decode throughput of a design (Ridotar, Fogezen, Fikizen, Zinizen, Mofidra) beside the Llama decoder at equal size.
+
+Mofidra: differential attention (two maps of 64 over values of 128 per head, as many heads and kv heads
+as the Llama model) beside the feed-forward in every layer; the first layer's feed-forward is dense,
+the others route every token to ``top`` of ``experts`` ungated experts beside a shared one; the second
+layer runs twice in a row, as many layer runs as the Llama model has layers.  It is also run beside
+Zinizen, the design closest to it (softmax attention and routed experts beside a shared one).
 
 Zinizen: layers cycling through the RG-LRU block, biased capped attention that shares values between
 its layers, gated latent attention and the biased attention once more; the first layer's feed-forward
@@ -125,9 +131,22 @@ def zinizen_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 33, "mul_cur": 5}}, "layers": out}
 
 
-DESIGNS = {"ridotar": ridotar_config, "fogezen": fogezen_config, "fikizen": fikizen_config, "zinizen": zinizen_config}
+def mofidra_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:
+    heads = width // 128
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff}}
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.6,
+                 "rot": {"base": 10000.0, "dims": 64}}
+    out = [{"type": "attention", "mixer": dict(attention), "mlp": {"kind": "dense", "ff": top * ff} if i == 0 else moe}
+           for i in range(max(2, layers - 1))]
+    return {"architecture": "Mofidra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"scale": float(width) ** 0.5}, "layers": out,
+            "loop": {"start": 1, "stop": 2, "times": 2 if layers > 2 else 1}}
+
+
+DESIGNS = {"ridotar": ridotar_config, "fogezen": fogezen_config, "fikizen": fikizen_config, "zinizen": zinizen_config,
+           "mofidra": mofidra_config}
 # the designs each is also measured beside (Llama always is)
-CLOSEST = {"fikizen": ("fogezen",), "zinizen": ("ridotar",)}
+CLOSEST = {"fikizen": ("fogezen",), "zinizen": ("ridotar",), "mofidra": ("zinizen",)}
 
 
 def llama_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:
