@@ -1491,7 +1491,8 @@ def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, ca
     ``attention_dv``.
 
     bfloat16 with both sizes multiples of 8 (dk up to 128, dv up to 256) runs on the tensor cores; everything
-    else runs the generic kernel.  Single tokens that stand before a step's portions (as the scheduler puts
+    else runs the generic kernel.  Portions of 128 tokens and more with dv up to 128 and no chunks go to the tcgen05
+    prompt kernel.  Single tokens that stand before a step's portions (as the scheduler puts
     them) get a launch of their own, shaped for rows that wait on memory."""
     _req(q, "q", dim=2)
     _req(out, "out", q.dtype, 2)
@@ -1520,6 +1521,14 @@ def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, ca
             spans = [(0, first, 1), (first, ctx.n_requests - first, ctx.max_q_len)]
     sms = num_sms(q.device)
     for at, n_req, max_q in spans:
+        if (max_q >= 128 and not chunk and USE_TCGEN05_ATTENTION and _lib("attention_diff_tc5").lsb_prefill_attention_diff_tc5_supported(
+                _p(q), _p(cache.k_pages), _p(cache.v_pages), _p(out), _i(nh), _i(nkv), _i(dk), _i(dv), _i(cache.page_size),
+                _f(scale))):
+            _call("attention_diff_tc5", "lsb_prefill_attention_diff_tc5", _p(q), _i(T), _p(cache.k_pages), _p(cache.v_pages),
+                  ctypes.c_void_p(ctx.q_start.data_ptr() + 4 * at), ctypes.c_void_p(ctx.kv_len.data_ptr() + 4 * at),
+                  ctypes.c_void_p(ctx.table_rows.data_ptr() + 4 * at), *common, _i(n_req), _i(max_q), *sizes[:7], _i(window),
+                  *sizes[9:], _stream(out))
+            continue
         plan = lib.lsb_attention_diff_plan(_i(n_req), _i(max_q), _i(nh), _i(nkv), _i(chunk), _i(sms), _i(DV_BLOCK_SHAPE))
         scratch = None
         if plan >> 8 > 1:

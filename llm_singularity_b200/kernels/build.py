@@ -49,6 +49,7 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     "attention_prep": "attention_prep.cu",
     "attention_dv": "attention_dv.cu",
     "attention_diff": "attention_diff.cu",
+    "attention_diff_tc5": "attention_diff_tc5.cu",
     "matrix_memory": "matrix_memory.cu",
     "delta_rule": "delta_rule.cu",
     "rglru": "rglru.cu",
@@ -57,7 +58,7 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     # host code only: pools, block tables, prefix tree; scheduler
     "host_runtime": ("host_memory.cpp", "host_scheduler.cpp", "host_step.cpp"),
 }
-HEADERS = ["common.cuh", "attention_tc_noalloc.h", "attention_dv.cuh", "stream_warm.cuh"]     # of the CUDA libraries
+HEADERS = ["common.cuh", "attention_tc_noalloc.h", "attention_dv.cuh", "attention_tc5.cuh", "stream_warm.cuh"]     # of the CUDA libraries
 HOST_HEADERS = ["host_memory.h"]                          # of the host runtime
 
 

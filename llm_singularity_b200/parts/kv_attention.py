@@ -79,6 +79,8 @@ class KVAttention(Part):
                       and 16 <= s.key_dim <= 256 and self.diff is None and not self.sink and not self.softcap and not self.linear_bias)
         if self.diff is not None:
             self.kernels = ("gemm", "attention_prep", "attention_diff")
+            if rt.dtype == torch.bfloat16 and s.chunk is None:
+                self.kernels = self.kernels + ("attention_diff_tc5",)
         elif self.plain:
             self.kernels = self.kernels + ("attention",)
             if rt.dtype == torch.bfloat16 and s.key_dim in (64, 128):
