@@ -20,6 +20,7 @@
 // requests bring at most 16 rows each get blocks of 16 rows, the four warps of a map dealing the keys of
 // a tile among themselves; where such blocks are few, a row tile's keys are shared among up to eight
 // blocks whose partial sums a second kernel brings together.
+#define LSB_CLUSTER_ALONG_X
 #include "attention_dv.cuh"
 
 LSB_DEFINE_STATUS()
@@ -466,6 +467,418 @@ attention_diff_mma_kernel(const DiffArgs a, float scale_log2, int ksplit, float*
     }
 }
 
+// ------------------------------------------------------------------ rows that wait on memory
+// Steps whose requests bring at most 16 rows each (single tokens: one row per query head of a kv head's
+// group), values of up to 128.  A block owns a request, a kv head and 16 rows; its four warps walk the keys
+// on their own, 16 at a time, each with a ring of its own in shared memory, so that no warp waits for
+// another until the end.  A warp holds both maps: a chunk's values are read from shared memory once for
+// both.  Chunks that hold cached keys only are asked for before the wait on the previous kernel (the
+// step's metadata and the block table are in place by then).  The blocks that share a row tile's keys are
+// one cluster: each leaves its sums in its shared memory, and after the cluster has met, each brings
+// its share of the rows together.  LOW8: at most 8 rows, the lower half of every fragment is left alone.
+constexpr int kDecWarps = 4, kDecKeys = 16;
+
+template <int DKP, int DVP>
+struct DecTile {
+    static constexpr int STAGES = DKP == 64 ? 3 : 2;
+    static constexpr int KS = 2 * DKP + 8, VS = DVP + 8;    // row strides in elements: 4 words past a multiple of 32
+    static constexpr int PS = DVP + 2;                      // a row of sums: O, then m and l
+    static constexpr int kStage = kDecKeys * (KS + VS);     // elements of a warp's chunk
+    static constexpr size_t kRing = (size_t)kDecWarps * STAGES * kStage * 2;
+    static constexpr size_t kMeet = (size_t)(kDecWarps + 1) * 16 * 2 * PS * 4;
+    static constexpr size_t kTotal = kRing > kMeet ? kRing : kMeet;
+};
+
+__device__ __forceinline__ float diff_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float ld_peer(const float* p, uint32_t rank) {
+    uint32_t peer;
+    float v;
+    asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(peer) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(peer) : "memory");
+    return v;
+}
+__device__ __forceinline__ void cluster_meet() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+template <int DKP, int DVP, bool LOW8>
+__global__ void __launch_bounds__(kDecWarps * 32, 2)
+attention_diff_decode_kernel(const DiffArgs a, float scale_log2, int ksplit) {
+    using L = DecTile<DKP, DVP>;
+    typedef __nv_bfloat16 bf16;
+    constexpr int KS = L::KS, VS = L::VS, PS = L::PS, ST = L::STAGES, NB = DVP / 8, NC = DVP / 32;
+    extern __shared__ __align__(16) unsigned char diff_smem[];
+    lsb_pdl_launch_dependents();
+    const int nh = a.nh, nkv = a.nkv, dk = a.dk, dv = a.dv, page_size = a.page_size;
+    const int r = blockIdx.z, g = blockIdx.y, group = nh / nkv;
+    const int qs = a.q_start[r];
+    const int q_len = a.q_start[r + 1] - qs;
+    const int rows_total = q_len * group;
+    const int row_tile = blockIdx.x / ksplit, part_id = blockIdx.x % ksplit;
+    const int tile_row0 = row_tile * 16;
+    if (tile_row0 >= rows_total) return;               // (every block of a cluster leaves here, or none)
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tid4 = lane & 3;
+    const int p_base = a.kv_len[r] - q_len;
+    const int rows_here = min(16, rows_total - tile_row0);
+    const int last_pos = p_base + (tile_row0 + rows_here - 1) / group;
+    const int first_pos = p_base + tile_row0 / group;
+    const int key_lo = diff_lowest(first_pos, a.window, a.chunk);      // the first key any row of the block sees
+    const int last_lo = diff_lowest(last_pos, a.window, a.chunk);
+    int c0 = key_lo / kDecKeys, c1 = last_pos / kDecKeys + 1;
+    {                                                  // this block's share of the chunks (it may be empty)
+        const int per = (c1 - c0 + ksplit - 1) / ksplit;
+        c0 += part_id * per;
+        c1 = min(c1, c0 + per);
+    }
+    const int n = max(0, (c1 - c0 - warp + kDecWarps - 1) / kDecWarps);      // chunks c0 + warp, + 4, ...
+    const int* bt = a.block_table + (size_t)a.table_rows[r] * a.table_stride;
+    bf16* ring = reinterpret_cast<bf16*>(diff_smem) + warp * ST * L::kStage;
+    // the padding of the rows is zeroed once; copies never touch it
+    if (dk < DKP || dv < DVP) {
+        for (int row = lane; row < ST * kDecKeys; row += 32) {
+            bf16* kd = ring + (row / kDecKeys) * L::kStage + (row % kDecKeys) * KS;
+            bf16* vd = ring + (row / kDecKeys) * L::kStage + kDecKeys * KS + (row % kDecKeys) * VS;
+            for (int c = dk; c < DKP; ++c) kd[c] = kd[DKP + c] = __float2bfloat16_rn(0.f);
+            for (int c = dv; c < DVP; ++c) vd[c] = __float2bfloat16_rn(0.f);
+        }
+        __syncwarp();
+    }
+    // A chunk's copies: the warp takes a key at a time, a lane 16 bytes of the key's rows (first the keys of
+    // both maps, then the values).  A chunk's place is looked up a chunk ahead of the copies.  Pages of a
+    // multiple of 16 keys hold a chunk whole, its rows one after the other (rows past the last key and
+    // before the first are then copied too: they are finite and masked); other pages go key by key.
+    constexpr int kIter = (2 * DKP / 8 + DVP / 8 + 31) / 32;
+    const bool whole = page_size % kDecKeys == 0;
+    const int kper = dk >> 3, nk = 2 * kper, nv = dv >> 3;
+    const char* src0[kIter];                           // this lane's 16 bytes of row 0 of the pages
+    int src_step[kIter], dst_step[kIter];              // bytes from row to row there, and in the ring
+    uint32_t dst0[kIter];
+    bool mine[kIter];
+#pragma unroll
+    for (int u = 0; u < kIter; ++u) {
+        const int c = lane + 32 * u;
+        const bool is_k = c < nk;
+        mine[u] = c < nk + nv;
+        src0[u] = is_k ? (const char*)a.k_pages + c * 16 : (const char*)a.v_pages + (c - nk) * 16;
+        src_step[u] = (is_k ? 2 * dk : dv) * 2;
+        dst0[u] = (uint32_t)__cvta_generic_to_shared(ring) +
+                  2u * (uint32_t)(is_k ? (c >= kper ? DKP + (c - kper) * 8 : c * 8) : kDecKeys * KS + (c - nk) * 8);
+        dst_step[u] = (is_k ? KS : VS) * 2;
+    }
+    constexpr int kBad = -2, kNone = -1;
+    auto place = [&](int k) -> int {                   // (not looked at before the copies of a later turn)
+        const int key = (c0 + warp + k * kDecWarps) * kDecKeys + (whole ? 0 : lane & 15);
+        if (k >= n || (!whole && (key > last_pos || key < key_lo))) return kNone;
+        const int page = bt[key / page_size];
+        return page < 0 ? kBad : page;
+    };
+    auto issue = [&](int page, int k, int st) {
+        const int key = (c0 + warp + k * kDecWarps) * kDecKeys + (whole ? 0 : lane & 15);
+        long long at = -1;
+        if (page >= a.num_pages || page == kBad) lsb_set_status(LSB_BAD_PAGE);
+        else if (page >= 0) at = ((long long)page * nkv + g) * page_size + key % page_size;
+        if (whole) {
+            const int size = at >= 0 ? 16 : 0;         // (0: filled with zeros)
+            const long long row = at >= 0 ? at : 0;
+#pragma unroll
+            for (int u = 0; u < kIter; ++u) {
+                if (mine[u]) {
+                    const char* src = src0[u] + row * src_step[u];
+                    uint32_t dst = dst0[u] + (uint32_t)(st * L::kStage * 2);
+#pragma unroll
+                    for (int i = 0; i < kDecKeys; ++i) {
+                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(size) : "memory");
+                        src += src_step[u];
+                        dst += dst_step[u];
+                    }
+                }
+            }
+            return;
+        }
+#pragma unroll 1
+        for (int i = 0; i < kDecKeys; ++i) {
+            const long long row = __shfl_sync(0xffffffffu, at, i);
+            const int size = row >= 0 ? 16 : 0;
+#pragma unroll
+            for (int u = 0; u < kIter; ++u)
+                if (mine[u])
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;"
+                                 ::"r"(dst0[u] + (uint32_t)(st * L::kStage * 2 + i * dst_step[u])),
+                                   "l"(src0[u] + (row >= 0 ? row * src_step[u] : 0)), "r"(size) : "memory");
+        }
+    };
+    auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+    int pages[ST - 1];
+#pragma unroll
+    for (int st = 0; st < ST - 1; ++st) pages[st] = place(st);
+    // chunks of keys that earlier steps cached do not depend on the kernel before
+    int early = 0;
+#pragma unroll
+    for (int st = 0; st < ST - 1; ++st)
+        if (st < n && (c0 + warp + st * kDecWarps + 1) * kDecKeys <= p_base) early = st + 1;
+#pragma unroll
+    for (int st = 0; st < ST - 1; ++st) {
+        if (st < early) {
+            issue(pages[st], st, st);
+            commit();
+        }
+    }
+    int at_next = place(ST - 1);
+    lsb_pdl_wait();
+#pragma unroll
+    for (int st = 0; st < ST - 1; ++st) {
+        if (st >= early) {
+            if (st < n) issue(pages[st], st, st);
+            commit();
+        }
+    }
+
+    // this thread's two rows (gid and gid + 8)
+    const int row_a = tile_row0 + gid, row_b = row_a + 8;
+    const bool ok_a = row_a < rows_total, ok_b = !LOW8 && row_b < rows_total;
+    const int pos_a = p_base + row_a / group, pos_b = p_base + row_b / group;
+    const int lo_a = diff_lowest(pos_a, a.window, a.chunk), lo_b = diff_lowest(pos_b, a.window, a.chunk);
+    uint32_t qa[2][DKP / 16][4];
+    {
+        const bf16* qa_row = (const bf16*)a.q + (((size_t)qs + row_a / group) * nh + g * group + row_a % group) * (2 * dk);
+        const bf16* qb_row = (const bf16*)a.q + (((size_t)qs + row_b / group) * nh + g * group + row_b % group) * (2 * dk);
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+#pragma unroll
+            for (int ks = 0; ks < DKP / 16; ++ks) {
+                uint32_t(&f)[4] = qa[mp][ks];
+                f[0] = f[1] = f[2] = f[3] = 0u;
+                const int c = mp * dk + ks * 16 + 2 * tid4;
+                if (ks * 16 < dk) {
+                    if (ok_a) f[0] = *reinterpret_cast<const uint32_t*>(qa_row + c);
+                    if (ok_b) f[1] = *reinterpret_cast<const uint32_t*>(qb_row + c);
+                }
+                if (ks * 16 + 8 < dk) {
+                    if (ok_a) f[2] = *reinterpret_cast<const uint32_t*>(qa_row + c + 8);
+                    if (ok_b) f[3] = *reinterpret_cast<const uint32_t*>(qb_row + c + 8);
+                }
+            }
+        }
+    }
+    float o[2][NB][4];
+    float m_a[2], m_b[2], l_a[2], l_b[2];
+#pragma unroll
+    for (int mp = 0; mp < 2; ++mp) {
+        m_a[mp] = m_b[mp] = -FLT_MAX;
+        l_a[mp] = l_b[mp] = 0.f;
+#pragma unroll
+        for (int nb = 0; nb < NB; ++nb) o[mp][nb][0] = o[mp][nb][1] = o[mp][nb][2] = o[mp][nb][3] = 0.f;
+    }
+    for (int k = 0; k < n; ++k) {
+        if (k + ST - 1 < n) issue(at_next, k + ST - 1, (k + ST - 1) % ST);
+        commit();                                      // (a group a turn, real or not)
+        at_next = place(k + ST);
+        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 1) : "memory");
+        __syncwarp();
+        const bf16* kb = ring + (k % ST) * L::kStage;
+        const int key0 = (c0 + warp + k * kDecWarps) * kDecKeys;
+        const bool interior = key0 >= last_lo && key0 + kDecKeys - 1 <= first_pos;
+        uint32_t pa[2][4];
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            const uint32_t kaddr = (uint32_t)__cvta_generic_to_shared(kb + ((lane & 7) + (lane >> 4) * 8) * KS + mp * DKP + ((lane >> 3) & 1) * 8);
+#pragma unroll
+            for (int ks = 0; ks < DKP / 16; ++ks) {
+                uint32_t b[4];
+                asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                             : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(kaddr + ks * 32));
+                dv_mma_16816(s[0], qa[mp][ks], b[0], b[1]);
+                dv_mma_16816(s[1], qa[mp][ks], b[2], b[3]);
+            }
+            constexpr int NE = LOW8 ? 2 : 4;
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+#pragma unroll
+                for (int e = 0; e < NE; ++e) s[j][e] *= scale_log2;
+            }
+            if (!interior) {
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+#pragma unroll
+                    for (int e = 0; e < NE; ++e) {
+                        const int key = key0 + j * 8 + 2 * tid4 + (e & 1);
+                        if (e < 2 ? (key < lo_a || key > pos_a) : (key < lo_b || key > pos_b)) s[j][e] = -INFINITY;
+                    }
+                }
+            }
+            float mx_a = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1])), mx_b = -FLT_MAX;
+            if (!LOW8) mx_b = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
+            mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
+            mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
+            if (!LOW8) {
+                mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
+                mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
+            }
+            // accumulators are rescaled only when a maximum has moved
+            if (__any_sync(0xffffffffu, mx_a > m_a[mp] || (!LOW8 && mx_b > m_b[mp]))) {
+                const float mn_a = fmaxf(m_a[mp], mx_a), corr_a = diff_exp2(m_a[mp] - mn_a);
+                m_a[mp] = mn_a;
+                l_a[mp] *= corr_a;
+#pragma unroll
+                for (int nb = 0; nb < NB; ++nb) {
+                    o[mp][nb][0] *= corr_a;
+                    o[mp][nb][1] *= corr_a;
+                }
+                if (!LOW8) {
+                    const float mn_b = fmaxf(m_b[mp], mx_b), corr_b = diff_exp2(m_b[mp] - mn_b);
+                    m_b[mp] = mn_b;
+                    l_b[mp] *= corr_b;
+#pragma unroll
+                    for (int nb = 0; nb < NB; ++nb) {
+                        o[mp][nb][2] *= corr_b;
+                        o[mp][nb][3] *= corr_b;
+                    }
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+#pragma unroll
+                for (int e = 0; e < NE; ++e) {
+                    // (a masked score is -inf and no maximum ever is: its weight is 0)
+                    const float pv = diff_exp2(s[j][e] - (e < 2 ? m_a[mp] : m_b[mp]));
+                    s[j][e] = pv;
+                    if (e < 2) l_a[mp] += pv;
+                    else l_b[mp] += pv;
+                }
+                pa[mp][2 * j] = dv_pack(s[j][0], s[j][1]);
+                pa[mp][2 * j + 1] = LOW8 ? 0u : dv_pack(s[j][2], s[j][3]);
+            }
+        }
+        const uint32_t vaddr = (uint32_t)__cvta_generic_to_shared(kb + kDecKeys * KS + (lane & 15) * VS + (lane >> 4) * 8);
+#pragma unroll
+        for (int nb = 0; nb < NB; nb += 2) {
+            uint32_t b[4];
+            asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                         : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(vaddr + nb * 16));
+#pragma unroll
+            for (int mp = 0; mp < 2; ++mp) {
+                dv_mma_16816(o[mp][nb], pa[mp], b[0], b[1]);
+                dv_mma_16816(o[mp][nb + 1], pa[mp], b[2], b[3]);
+            }
+        }
+        __syncwarp();                                  // the chunk's buffer may be filled again
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();
+    // the four warps' sums meet in shared memory
+    float* part = reinterpret_cast<float*>(diff_smem);       // [warp][row][map][PS]
+    float* comb = part + kDecWarps * 16 * 2 * PS;            // [row][map][PS]: the block's sums, for its cluster
+#pragma unroll
+    for (int mp = 0; mp < 2; ++mp) {
+        l_a[mp] += __shfl_xor_sync(0xffffffffu, l_a[mp], 1);
+        l_a[mp] += __shfl_xor_sync(0xffffffffu, l_a[mp], 2);
+        float* da = part + ((warp * 16 + gid) * 2 + mp) * PS;
+#pragma unroll
+        for (int nb = 0; nb < NB; ++nb) *reinterpret_cast<float2*>(&da[nb * 8 + 2 * tid4]) = make_float2(o[mp][nb][0], o[mp][nb][1]);
+        if (tid4 == 0) {
+            da[DVP] = m_a[mp];
+            da[DVP + 1] = l_a[mp];
+        }
+        if (!LOW8) {
+            l_b[mp] += __shfl_xor_sync(0xffffffffu, l_b[mp], 1);
+            l_b[mp] += __shfl_xor_sync(0xffffffffu, l_b[mp], 2);
+            float* db = da + 8 * 2 * PS;
+#pragma unroll
+            for (int nb = 0; nb < NB; ++nb) *reinterpret_cast<float2*>(&db[nb * 8 + 2 * tid4]) = make_float2(o[mp][nb][2], o[mp][nb][3]);
+            if (tid4 == 0) {
+                db[DVP] = m_b[mp];
+                db[DVP + 1] = l_b[mp];
+            }
+        }
+    }
+    __syncthreads();
+    const float lambda = a.lambda[0];
+    auto finish = [&](float (&y)[2][NC], const float (&den)[2], int row_l) {
+        const float i0 = den[0] > 0.f ? 1.f / den[0] : 0.f, i1 = den[1] > 0.f ? lambda / den[1] : 0.f;
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            y[0][c] = y[0][c] * i0 - y[1][c] * i1;           // (zero past dv)
+            ss += y[0][c] * y[0][c];
+        }
+        const float mul = a.post / sqrtf(lsb_warp_sum(ss) / (float)dv + a.eps);
+        const int row = tile_row0 + row_l;
+        bf16* dst = (bf16*)a.out + (((size_t)qs + row / group) * nh + g * group + row % group) * dv;
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+            if (lane + 32 * c < dv) dst[lane + 32 * c] = __float2bfloat16_rn(y[0][c] * mul);
+    };
+    for (int row_l = warp; row_l < rows_here; row_l += kDecWarps) {      // a warp brings a row together
+        float y[2][NC], den[2];
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+            const float* src = part + (row_l * 2 + mp) * PS;
+            constexpr int WS = 16 * 2 * PS;
+            float mm = -FLT_MAX, f[kDecWarps];
+            den[mp] = 0.f;
+#pragma unroll
+            for (int w = 0; w < kDecWarps; ++w) mm = fmaxf(mm, src[w * WS + DVP]);
+#pragma unroll
+            for (int w = 0; w < kDecWarps; ++w) {
+                f[w] = exp2f(src[w * WS + DVP] - mm);
+                den[mp] += f[w] * src[w * WS + DVP + 1];
+            }
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                y[mp][c] = 0.f;
+#pragma unroll
+                for (int w = 0; w < kDecWarps; ++w) y[mp][c] += f[w] * src[w * WS + lane + 32 * c];
+            }
+            if (ksplit > 1) {
+                float* dst = comb + (row_l * 2 + mp) * PS;
+#pragma unroll
+                for (int c = 0; c < NC; ++c) dst[lane + 32 * c] = y[mp][c];
+                if (lane == 0) {
+                    dst[DVP] = mm;
+                    dst[DVP + 1] = den[mp];
+                }
+            }
+        }
+        if (ksplit == 1) finish(y, den, row_l);
+    }
+    if (ksplit == 1) return;
+    cluster_meet();
+    for (int row_l = part_id * kDecWarps + warp; row_l < rows_here; row_l += ksplit * kDecWarps) {
+        float y[2][NC], den[2];
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+            const float* src = comb + (row_l * 2 + mp) * PS;
+            float f[kMaxParts], l[kMaxParts], v[kMaxParts][NC], mm = -FLT_MAX;
+#pragma unroll
+            for (int p = 0; p < kMaxParts; ++p) {            // all peers' values in flight at once
+                f[p] = p < ksplit ? ld_peer(src + DVP, p) : -FLT_MAX;
+                l[p] = p < ksplit ? ld_peer(src + DVP + 1, p) : 0.f;
+#pragma unroll
+                for (int c = 0; c < NC; ++c) v[p][c] = p < ksplit ? ld_peer(src + lane + 32 * c, p) : 0.f;
+            }
+#pragma unroll
+            for (int p = 0; p < kMaxParts; ++p) mm = fmaxf(mm, f[p]);
+            den[mp] = 0.f;
+#pragma unroll
+            for (int c = 0; c < NC; ++c) y[mp][c] = 0.f;
+#pragma unroll
+            for (int p = 0; p < kMaxParts; ++p) {            // summed in rank order
+                const float w = p < ksplit ? exp2f(f[p] - mm) : 0.f;
+                den[mp] += w * l[p];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) y[mp][c] += w * v[p][c];
+            }
+        }
+        finish(y, den, row_l);
+    }
+    cluster_meet();                                    // nobody leaves while a peer may still read its shared memory
+}
+
 // The partial sums of `ksplit` blocks that shared a row tile's keys, brought together, differenced and
 // normed: scratch [request, kv head, row tile, part, 16 rows, map, dv + 2].  A warp owns a row.
 template <int NC>
@@ -527,9 +940,24 @@ attention_diff_merge_kernel(const float* __restrict__ scratch, const DiffArgs a,
 }
 
 // ------------------------------------------------------------------ host side
-// See dv_mma_plan: 16-row blocks or not, tiles in flight, blocks that share a row tile's keys.
-LSB_API int lsb_attention_diff_plan(int n_requests, int max_q_len, int nh, int nkv, int chunk, int sms, int shape) {
-    return dv_mma_plan(n_requests, max_q_len, nh, nkv, chunk, sms, shape);
+// How a step of this shape is launched, as dv_mma_plan says (16-row blocks or not, tiles in flight, blocks that
+// share a row tile's keys); bit 2: the kernel whose warps walk the keys on their own, for steps of at
+// most 16 rows a request and values of up to 128.  shape 5 and more: that kernel with keys shared by
+// shape - 4 blocks; 1 - 4 as in dv_mma_plan.
+static int diff_plan(int n_requests, int max_q_len, int nh, int nkv, int dv, int chunk, int sms, int shape) {
+    const long long rows = (long long)max_q_len * (nh / nkv);
+    if (dv > 128 || (shape == 0 && rows > 16) || (shape >= 1 && shape <= 4))
+        return dv_mma_plan(n_requests, max_q_len, nh, nkv, chunk, sms, shape > 4 ? 0 : shape);
+    if (sms <= 0) sms = 148;
+    const long long thin = (rows + 15) / 16 * nkv * n_requests;
+    long long ksplit = shape > 4 ? shape - 4 : (2 * sms) / thin;       // two blocks fit an SM
+    if (ksplit > kMaxParts) ksplit = kMaxParts;
+    if (shape == 0 && chunk > 0 && ksplit > (chunk + kMmaKeys - 1) / kMmaKeys) ksplit = (chunk + kMmaKeys - 1) / kMmaKeys;
+    if (ksplit < 1) ksplit = 1;
+    return 4 | ((int)ksplit << 8);
+}
+LSB_API int lsb_attention_diff_plan(int n_requests, int max_q_len, int nh, int nkv, int dv, int chunk, int sms, int shape) {
+    return diff_plan(n_requests, max_q_len, nh, nkv, dv, chunk, sms, shape);
 }
 
 LSB_API int lsb_attention_diff_mma_supported(int dk, int dv) {
@@ -572,6 +1000,24 @@ static int launch_shape(const DiffArgs& a, int plan, dim3 grid, float* scratch, 
                     : launch_mma<DKP, DVP, 2, true>(a, grid, ksplit, scratch, stream);
 }
 
+template <int DKP, int DVP, bool LOW8>
+static int launch_decode_rows(const DiffArgs& a, dim3 grid, int ksplit, cudaStream_t stream) {
+    constexpr size_t smem = DecTile<DKP, DVP>::kTotal;
+    static_assert(2 * (smem + 1024) <= 228 * 1024, "two blocks an SM");
+    static int configured = -1;
+    if (configured < 0)
+        configured = (int)cudaFuncSetAttribute(attention_diff_decode_kernel<DKP, DVP, LOW8>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (configured) return configured;
+    return lsb_launch(attention_diff_decode_kernel<DKP, DVP, LOW8>, grid, dim3(kDecWarps * 32), smem, stream, ksplit, a,
+                      a.scale * 1.4426950408889634f, ksplit);
+}
+
+template <int DKP, int DVP>
+static int launch_decode(const DiffArgs& a, dim3 grid, int ksplit, bool low8, cudaStream_t stream) {
+    return low8 ? launch_decode_rows<DKP, DVP, true>(a, grid, ksplit, stream) : launch_decode_rows<DKP, DVP, false>(a, grid, ksplit, stream);
+}
+
 // bfloat16; q, the pages and out 16-byte aligned; sms: the device's multiprocessors (what a small grid is
 // measured against); scratch: n_requests * nkv * row tiles * parts * 16 * 2 * (dv + 2) floats if the plan has parts.
 LSB_API int lsb_attention_diff_mma(const void* q, const void* k_pages, const void* v_pages, const int* q_start,
@@ -586,7 +1032,12 @@ LSB_API int lsb_attention_diff_mma(const void* q, const void* k_pages, const voi
     const DiffArgs a = diff_args(q, k_pages, v_pages, q_start, kv_len, table_rows, block_table, table_stride, out, nh, nkv,
                                  dk, dv, page_size, num_pages, scale, window, chunk, lambda, eps, post);
     const long long rows = (long long)max_q_len * (nh / nkv);
-    const int plan = dv_mma_plan(n_requests, max_q_len, nh, nkv, chunk, sms, shape);
+    const int plan = diff_plan(n_requests, max_q_len, nh, nkv, dv, chunk, sms, shape);
+    if (plan & 4) {
+        const dim3 dgrid((unsigned)((rows + 15) / 16) * (plan >> 8), nkv, n_requests);
+        if (dk <= 64) return dv <= 64 ? launch_decode<64, 64>(a, dgrid, plan >> 8, rows <= 8, stream) : launch_decode<64, 128>(a, dgrid, plan >> 8, rows <= 8, stream);
+        return dv <= 64 ? launch_decode<128, 64>(a, dgrid, plan >> 8, rows <= 8, stream) : launch_decode<128, 128>(a, dgrid, plan >> 8, rows <= 8, stream);
+    }
     const int ksplit = plan >> 8;
     if (ksplit > 1 && !scratch) return (int)cudaErrorInvalidValue;
     const unsigned tiles = (unsigned)(plan & 1 ? (rows + 15) / 16 : (rows + kMmaRows - 1) / kMmaRows);

@@ -1529,9 +1529,10 @@ def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, ca
                   ctypes.c_void_p(ctx.table_rows.data_ptr() + 4 * at), *common, _i(n_req), _i(max_q), *sizes[:7], _i(window),
                   *sizes[9:], _stream(out))
             continue
-        plan = lib.lsb_attention_diff_plan(_i(n_req), _i(max_q), _i(nh), _i(nkv), _i(chunk), _i(sms), _i(DV_BLOCK_SHAPE))
+        plan = lib.lsb_attention_diff_plan(_i(n_req), _i(max_q), _i(nh), _i(nkv), _i(dv), _i(chunk), _i(sms),
+                                           _i(DV_BLOCK_SHAPE))
         scratch = None
-        if plan >> 8 > 1:
+        if plan >> 8 > 1 and not plan & 4:
             tiles = -(-max_q * (nh // nkv) // 16)
             key = ("attention_diff", q.device, n_req * nkv * tiles * (plan >> 8) * 16 * 2 * (dv + 2))
             scratch = _scratch.get(key)
