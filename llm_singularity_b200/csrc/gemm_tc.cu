@@ -162,6 +162,8 @@ struct GemmParams {
     // earlier in the stream, so a block reads it only after the wait on that kernel.
     const int* tile_group;
     int group_rows;
+    // Swapped: P stacks the groups' matrices and tile_group[j0 / BN] names the group of a BN-row tile of Q.
+    int group_swap;
 };
 
 template <int BN>
@@ -365,7 +367,7 @@ __device__ __forceinline__ void epilogue_staged(const GemmParams& prm, unsigned 
 // now), the four epilogue warps meet, and each output row leaves as one 128-byte run.
 template <int BN>
 __device__ __forceinline__ void epilogue_swap_gated(const GemmParams& prm, unsigned char* stage_base,
-                                                    uint32_t tmem_base, int q, int lane, int i0,
+                                                    uint32_t tmem_base, int q, int lane, int i0, int j0,
                                                     const int* abort_flag) {
     bf16* tile = reinterpret_cast<bf16*>(stage_base);         // [BN][64]
     const int n_local = (q * 32 + lane) >> 1;                 // this pair's output among the tile's 64
@@ -389,10 +391,10 @@ __device__ __forceinline__ void epilogue_swap_gated(const GemmParams& prm, unsig
     const int t = q * 32 + lane;
     bf16* out = reinterpret_cast<bf16*>(prm.out);
     for (int idx = t; idx < BN * 8; idx += 128) {              // 16-byte chunks: eight a batch row
-        const int m = idx >> 3, c = idx & 7;
+        const int m = j0 + (idx >> 3), c = idx & 7;
         if (m < prm.rows_q && n0 + c * 8 < n_out)
             *reinterpret_cast<uint4*>(out + (long long)m * prm.ldc_j + n0 + c * 8) =
-                *reinterpret_cast<const uint4*>(tile + m * 64 + c * 8);
+                *reinterpret_cast<const uint4*>(tile + (idx >> 3) * 64 + c * 8);
     }
 }
 
@@ -431,12 +433,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
     const int nkb = max(0, kb1 - kb0);
 
     lsb_pdl_launch_dependents();
-    int jq0 = j0;                                  // first row of this tile's Q operand
+    int ip0 = i0, jq0 = j0;                        // first rows of this tile's operands
     if (prm.tile_group) {
         lsb_pdl_wait();
-        const int g = prm.tile_group[blockIdx.x];
+        const int g = prm.tile_group[prm.group_swap ? blockIdx.y : blockIdx.x];
         if (g < 0) return;                         // (before any barrier or tensor memory exists)
-        jq0 = j0 + g * prm.group_rows;
+        if (prm.group_swap) ip0 = i0 + g * prm.group_rows;
+        else jq0 = j0 + g * prm.group_rows;
     }
     const int pre = min(nkb, STAGES);
     if (threadIdx.x == 0) {
@@ -451,7 +454,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
         for (int kb = 0; kb < pre; ++kb) {
             unsigned char* st = stages + (size_t)kb * L::kStageBytes;
             mbar_expect_tx(&full[kb], L::kStageBytes);
-            if (prm.static_operand == 1) tma_load_2d(st, &map_p, &full[kb], (kb0 + kb) * kBK, i0);
+            if (prm.static_operand == 1) tma_load_2d(st, &map_p, &full[kb], (kb0 + kb) * kBK, ip0);
             else tma_load_2d(st + L::kPBytes, &map_q, &full[kb], (kb0 + kb) * kBK, jq0);
         }
     }
@@ -468,7 +471,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
             for (int kb = 0; kb < pre; ++kb) {
                 unsigned char* st = stages + (size_t)kb * L::kStageBytes;
                 if (prm.static_operand == 1) tma_load_2d(st + L::kPBytes, &map_q, &full[kb], (kb0 + kb) * kBK, jq0);
-                else tma_load_2d(st, &map_p, &full[kb], (kb0 + kb) * kBK, i0);
+                else tma_load_2d(st, &map_p, &full[kb], (kb0 + kb) * kBK, ip0);
             }
             int issued = pre;
             for (int kb = pre; kb < nkb; ++kb) {
@@ -476,7 +479,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
                 if (!mbar_wait(&empty[s], ((kb / STAGES) - 1) & 1, &abort_flag)) break;
                 mbar_expect_tx(&full[s], L::kStageBytes);
                 unsigned char* st = stages + (size_t)s * L::kStageBytes;
-                tma_load_2d(st, &map_p, &full[s], (kb0 + kb) * kBK, i0);
+                tma_load_2d(st, &map_p, &full[s], (kb0 + kb) * kBK, ip0);
                 tma_load_2d(st + L::kPBytes, &map_q, &full[s], (kb0 + kb) * kBK, jq0);
                 issued = kb + 1;
             }
@@ -528,11 +531,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
                     epilogue_staged<BN, false>(prm, stages, tmem_base, q, lane, i0, j0);
                 }
             }
-        } else if (prm.splits == 1 && prm.swiglu == 2 && !prm.out_f32 && prm.ldc_i == 1 && nkb > 0 && j0 == 0 &&
+        } else if (prm.splits == 1 && prm.swiglu == 2 && !prm.out_f32 && prm.ldc_i == 1 && nkb > 0 &&
                    ((prm.rows_p >> 1) % 8) == 0 && (prm.ldc_j % 8) == 0 && (((uintptr_t)prm.out) & 15) == 0) {
             // (a condition on the parameters alone: all four warps go in, also after a wait that ran
             // out, because they meet inside; nothing is stored then)
-            epilogue_swap_gated<BN>(prm, stages, tmem_base, q, lane, i0, &abort_flag);
+            epilogue_swap_gated<BN>(prm, stages, tmem_base, q, lane, i0, j0, &abort_flag);
         } else if (prm.splits == 1) {
 #pragma unroll 1
             for (int c0 = 0; c0 < BN; c0 += 32) {
@@ -991,6 +994,7 @@ LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, in
     prm.limit = limit;
     prm.plain = plain;
     prm.tile_group = nullptr;
+    prm.group_swap = 0;
     prm.group_rows = 0;
     const int sms = num_sms();
     CUtensorMap mp, mq;
@@ -1073,16 +1077,18 @@ LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, in
 
 
 
-// Grouped form for routed experts: x [M, K] holds row tiles of 128 that belong to one group each
-// (tile_group[M / 128], device memory, -1 for an unused tile), w stacks `groups` matrices [N, K];
-// out[m] = x[m] w[group of m's tile]^T, gated (or with a plain activation) as above if swiglu.  M is a multiple of 128.
+// Grouped form for routed experts: x [M, K] holds row tiles of `tile` that belong to one group each
+// (tile_group[M / tile], device memory, -1 for an unused tile), w stacks `groups` matrices [N, K];
+// out[m] = x[m] w[group of m's tile]^T, gated (or with a plain activation) as above if swiglu.  M is a multiple of tile.
+// Tiles of 128 rows are the product's rows; tiles of 16, 32 or 64 (steps of few tokens, whose groups have a
+// few rows each) stand on the narrow side, the groups' matrices on the 128-row side.
 LSB_API int lsb_gemm_tc_grouped(const void* x, const void* w, void* out, int out_f32, int M, int N, int K,
-                                int groups, const int* tile_group, int swiglu, float limit, cudaStream_t stream) {
+                                int groups, const int* tile_group, int tile, int swiglu, float limit, cudaStream_t stream) {
     if (M <= 0) return 0;
     const int plain = swiglu >= LSB_PLAIN ? swiglu - LSB_PLAIN : 0;
     if (plain) swiglu = 0;
     if (plain && !known_plain(plain)) return (int)cudaErrorInvalidValue;
-    if (!lsb_gemm_tc_supported(x, w, M, N, K) || M % kBM || groups <= 0 || !tile_group) return (int)cudaErrorInvalidValue;
+    if (!lsb_gemm_tc_supported(x, w, M, N, K) || (tile != 16 && tile != 32 && tile != 64 && tile != kBM) || M % tile || groups <= 0 || !tile_group) return (int)cudaErrorInvalidValue;
     if ((swiglu && (N % 2)) || !known_act(swiglu)) return (int)cudaErrorInvalidValue;
     if ((long long)groups * N > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
     const int n_out = swiglu ? N / 2 : N;
@@ -1098,6 +1104,24 @@ LSB_API int lsb_gemm_tc_grouped(const void* x, const void* w, void* out, int out
     prm.plain = plain;
     prm.tile_group = tile_group;
     prm.group_rows = N;
+    prm.group_swap = tile < kBM ? 1 : 0;
+    if (tile < kBM) {
+        prm.rows_p = N; prm.rows_q = M; prm.ldc_i = 1; prm.ldc_j = n_out;
+        prm.swiglu = swiglu ? 2 : 0;
+        prm.static_operand = 1;
+        CUtensorMap sp, sq;
+        int src;
+        if ((src = make_map(&sp, w, groups * N, K, kBM))) return src;
+        if ((src = make_map(&sq, x, M, K, tile))) return src;
+        dim3 sgrid((N + kBM - 1) / kBM, M / tile, 1);
+        if (sgrid.y > 65535) return (int)cudaErrorInvalidValue;
+        // (a few stages, so that two or three blocks share an SM: there are a few more tiles than SMs)
+        switch (tile) {
+            case 16: return launch<16, 4>(sp, sq, prm, sgrid, stream);
+            case 32: return launch<32, 4>(sp, sq, prm, sgrid, stream);
+            default: return launch<64, 4>(sp, sq, prm, sgrid, stream);
+        }
+    }
     prm.rows_p = M; prm.rows_q = N; prm.ldc_i = n_out; prm.ldc_j = 1;
     prm.swiglu = swiglu ? 1 : 0;
     prm.static_operand = 2;

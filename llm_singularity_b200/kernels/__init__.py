@@ -1794,6 +1794,7 @@ def memory_output(walked: torch.Tensor, floor: torch.Tensor, weight: torch.Tenso
 # ------------------------------------------------------------------------ routed experts
 MOE_SCORES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
 MOE_TENSOR_CORES = True         # bfloat16 experts on the grouped tcgen05 product
+MOE_ROW_TILE = 0                # rows of its tiles: 16, 32, 64 or 128; 0: by the rows an expert gets
 
 
 def moe_tile() -> int:
@@ -1888,9 +1889,12 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     else:
         act = PRODUCT_PLAIN_ACTS[activation]
     # bfloat16 with TMA-friendly sizes: rows gathered in place, two grouped tcgen05 products over
-    # 128-row tiles; anything else (32-bit, odd sizes): the plain grouped kernels over 32-row tiles
+    # 128-row tiles, or over narrow ones where an expert gets a few rows; anything else (32-bit, odd sizes): the plain grouped kernels over 32-row tiles
     tc = MOE_TENSOR_CORES and x.dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0
-    tile = 128 if tc else moe_tile()
+    tile = moe_tile()
+    if tc:
+        mean = T * top / E                  # rows an expert gets
+        tile = MOE_ROW_TILE or (16 if mean <= 8 else 32 if mean <= 16 else 64 if mean <= 32 else 128)
     cap_tiles = -(-T * top // tile) + E
     dev = x.device
     pos = torch.empty(T * top, dtype=torch.int32, device=dev)
@@ -1914,9 +1918,9 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
               _i(cap_tiles * tile), _i(H), _p(rows), s)
         _chain_ends()
         _call("gemm_tc", "lsb_gemm_tc_grouped", _p(rows), _p(w_gate_up), _p(hidden), _i(0), _i(cap_tiles * tile),
-              _i(N_up), _i(H), _i(E), _p(tile_expert), _i(act if gated else _PLAIN + act), _f(limit), s)
+              _i(N_up), _i(H), _i(E), _p(tile_expert), _i(tile), _i(act if gated else _PLAIN + act), _f(limit), s)
         _call("gemm_tc", "lsb_gemm_tc_grouped", _p(hidden), _p(w_down), _p(y), _i(0), _i(cap_tiles * tile),
-              _i(H), _i(F), _i(E), _p(tile_expert), _i(0), _f(0.0), s)
+              _i(H), _i(F), _i(E), _p(tile_expert), _i(tile), _i(0), _f(0.0), s)
     else:
         _call("moe", "lsb_moe_up", _p(x), _i(_dt(x)), _p(row_token), _p(row_scale), _i(on_input), _p(w_gate_up),
               _p(tile_expert), _i(cap_tiles), _p(hidden), _i(F), _i(H), _i(act), _f(limit), _i(0 if gated else 1), s)

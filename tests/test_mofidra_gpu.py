@@ -416,6 +416,41 @@ def test_ungated_experts_beside_a_shared_one(dtype, T, W, F, E, top, S):
     assert (got - want).abs().max() < (1e-5 if dtype == torch.float32 else 5e-2) * max(1.0, scale), (got - want).abs().max()
 
 
+@pytest.mark.parametrize("tile", [16, 32, 64, 128])
+@pytest.mark.parametrize("act", ["relu_squared", "silu", "capped_glu"])
+@pytest.mark.parametrize("T, H, F, E, top", [(3, 64, 40, 4, 2), (150, 128, 136, 5, 3), (9, 72, 264, 9, 1)])
+def test_grouped_products_over_row_tiles_of_any_height(tile, act, T, H, F, E, top, monkeypatch):
+    """Experts gated and not, through both orientations of the grouped product; one expert gets more rows than a
+    tile, another none."""
+    from llm_singularity_b200 import kernels as K
+    monkeypatch.setattr(K, "MOE_ROW_TILE", tile)
+    g = torch.Generator().manual_seed(T + F)
+    gated, limit = act != "relu_squared", 0.9
+    bf = lambda *shape: (torch.randn(*shape, generator=g) / math.sqrt(shape[-1])).to(torch.bfloat16)
+    up, gate, down = bf(E, F, H), bf(E, F, H), bf(E, H, F)
+    x = torch.randn(T, H, generator=g).to(torch.bfloat16)
+    ids = torch.stack([torch.randperm(E - 1, generator=g)[:top] for _ in range(T)])          # the last expert idles
+    ids[:2 * T // 3, 0] = 1
+    wts = torch.rand(T, top, generator=g) + 0.2
+    want = torch.zeros(T, H, dtype=F64)
+    for t in range(T):
+        for k in range(top):
+            e = int(ids[t, k])
+            u, z = up[e].double() @ x[t].double(), gate[e].double() @ x[t].double()
+            if act == "capped_glu":
+                z = torch.clamp(z, max=limit)
+                hid = z * torch.sigmoid(1.702 * z) * (torch.clamp(u, -limit, limit) + 1.0)
+            else:
+                hid = z * torch.sigmoid(z) * u if gated else P.relu_squared(u)
+            want[t] += wts[t, k].double() * (down[e].double() @ hid)
+    w = torch.stack([gate, up], dim=2).reshape(E, 2 * F, H).contiguous() if gated else up
+    out = torch.empty(T, H, dtype=torch.bfloat16, device="cuda")
+    K.moe_experts(x.cuda(), ids.to(torch.int32).cuda(), wts.cuda(), w.cuda(), down.cuda(), act, "output", out, gated=gated,
+                  limit=limit if act == "capped_glu" else 0.0)
+    assert (out.double().cpu() - want).abs().max() < 3e-2 * max(1.0, want.abs().max())
+    K.check_status()
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("act", ["gelu_tanh", "relu_squared", "silu"])
 @pytest.mark.parametrize("M, K_, N", [(1, 64, 40), (9, 128, 300), (16, 192, 1000), (40, 128, 264), (100, 1024, 128), (300, 64, 520), (700, 72, 130),
