@@ -702,6 +702,32 @@ def _fork_join(ctx, device):
     return got
 
 
+OVERLAP_SUBLAYERS = 64          # steps of at most this many tokens run independent sublayers on two streams (0: none)
+_branch: Dict[torch.device, tuple] = {}
+
+
+def side_by_side(rows: int, device, first, second):
+    """(first(), second()), two chains of kernels that do not depend on one another: in a step of few rows, whose
+    kernels wait on memory and on one another, the second runs on a stream of its own beside the first.
+    What either allocates is used on its own stream until both have joined again, so that memory handed
+    back is only ever reused behind its last use."""
+    if _recording is not None or not 0 < rows <= OVERLAP_SUBLAYERS:
+        return first(), second()
+    got = _branch.get(device)
+    if got is None:
+        got = _branch[device] = (torch.cuda.Stream(device), torch.cuda.Event(), torch.cuda.Event())
+    side, fork, join = got
+    here = torch.cuda.current_stream(device)
+    fork.record(here)
+    side.wait_event(fork)
+    with torch.cuda.stream(side):
+        b = second()
+        join.record(side)
+    a = first()
+    here.wait_event(join)
+    return a, b
+
+
 def _batch_shape(ctx):
     """(single-token requests, first and one past the last request with more tokens) of a step;
     worked out once per step and kept on the context."""

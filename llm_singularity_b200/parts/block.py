@@ -100,10 +100,11 @@ class SideBySideBlock(Part):
 
     def forward(self, residual: torch.Tensor, pending, ctx, cache, writes_cache: bool = True):
         h = self.norm.add_norm(residual, pending)
-        y = self.mixer.forward(h, ctx, cache, writes_cache)
         if self.ffn is None:
-            return y
-        return DeltaPair(y, self.ffn.forward(h, ctx))
+            return self.mixer.forward(h, ctx, cache, writes_cache)
+        both = getattr(self.rt.ops, "side_by_side", None) or (lambda rows, device, first, second: (first(), second()))
+        return DeltaPair(*both(h.shape[0], h.device, lambda: self.mixer.forward(h, ctx, cache, writes_cache),
+                               lambda: self.ffn.forward(h, ctx)))
 
 
 class TokenSide(Part):

@@ -171,6 +171,29 @@ def test_long_decoding(tmp_path, dtype, name="mix_b"):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_sublayers_on_two_streams_give_the_same_bits(tmp_path, dtype, monkeypatch, name="mix_b"):
+    """A step of few rows runs mixer and feed-forward on two streams (captured in a graph and not): the same
+    bits as one after the other, over many steps whose buffers are reused."""
+    from llm_singularity_b200 import kernels as K
+    from llm_singularity_b200.engine.batch import StepEntry
+    cfg = U.CONFIGS[name]
+    W, path = _setup(tmp_path, cfg, 41)
+    toks = {k: U.tokens_for(cfg, 90, 50 + i) for i, k in enumerate("abc")}
+    got = []
+    for limit in (0, 64):
+        monkeypatch.setattr(K, "OVERLAP_SUBLAYERS", limit)
+        r = U.make_runner(path, dtype, pages=24)
+        assert all(r.open(k) for k in toks)
+        rows = [r.step([StepEntry(k, t[:20], [19]) for k, t in toks.items()]).float().cpu()]
+        rows += [r.step([StepEntry(k, t[i:i + 1], [0]) for k, t in toks.items()]).float().cpu() for i in range(20, 80)]
+        rows.append(r.step([StepEntry("b", toks["b"][80:], [9]), StepEntry("a", toks["a"][80:81], [0])]).float().cpu())
+        r.check_kernels()
+        assert r.graph_replays > 40
+        got.append(torch.cat(rows))
+    assert torch.equal(got[0], got[1])
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_greedy_generation_through_the_engine(tmp_path, dtype, name="mix_a"):
     """Greedy generation through Engine (scheduler, portions of 16, three requests at once) gives
     the tokens the plain model picks, wherever its choice is not a near tie."""
