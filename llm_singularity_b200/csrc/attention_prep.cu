@@ -259,6 +259,82 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
     }
 }
 
+// The common case without bias, norm, temperature or mixing, everything in whole 16 bytes (rotated dims in
+// "half" pairs, half of them a multiple of 16 bytes): a thread takes 16 bytes of a value, of a part of a
+// head that passes, or the two 16 bytes of a part of a head that turn together, straight from the
+// projection to its place.  One block per token; its sines and cosines are formed while the projection
+// before this kernel is still running.
+template <typename T>
+__global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_rotate_kernel(PrepArgs a) {
+    __shared__ float cs_sh[2][kPrepMaxDim / 2];
+    constexpr int VEC = PrepVec<T>::N;
+    lsb_pdl_launch_dependents();
+    const int t = blockIdx.x;
+    const int pos = a.positions[t];
+    const int half = a.rotary_dim >> 1;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &cs_sh[1][i], &cs_sh[0][i]);
+    const int slot_row = a.store ? a.table_rows[a.token_req[t]] : 0;      // (metadata too)
+    __syncthreads();
+    lsb_pdl_wait();
+    long long at = -1;                                   // (page, kv head 0, offset) as a row number
+    if (a.store) {
+        const int page_idx = pos / a.page_size;
+        int page = -1;
+        if (page_idx < a.table_stride) page = a.block_table[(size_t)slot_row * a.table_stride + page_idx];
+        if (page < 0 || page >= a.num_pages) {
+            if (threadIdx.x == 0) lsb_set_status(LSB_BAD_PAGE);
+        } else {
+            at = (long long)page * a.nkv * a.page_size + (pos % a.page_size);
+        }
+    }
+    const T* row = (const T*)a.proj + (size_t)t * a.ld;
+    const int nq = a.nh * a.maps, nk = a.nkv * a.maps;   // parts of heads
+    const int turning = half / VEC, per = turning + (a.dk - a.rotary_dim) / VEC;      // items of a part
+    const int items = (nq + nk) * per + a.nkv * a.dv / VEC;
+    for (int w = threadIdx.x; w < items; w += blockDim.x) {
+        if (w >= (nq + nk) * per) {                      // values
+            const int i = (w - (nq + nk) * per) * VEC, head = i / a.dv, d = i - head * a.dv;
+            const uint4 raw = *reinterpret_cast<const uint4*>(row + a.v_off + i);
+            if (at >= 0) *reinterpret_cast<uint4*>((T*)a.v_pages + (at + (long long)head * a.page_size) * a.dv + d) = raw;
+            continue;
+        }
+        const int part = w / per, j = w - part * per;
+        const bool is_q = part < nq;
+        const int hp = is_q ? part : part - nq;
+        const T* src = row + (is_q ? a.q_off : a.k_off) + hp * a.dk;
+        T* dst = nullptr;
+        if (is_q) dst = (T*)a.q_out + ((size_t)t * nq + hp) * a.dk;
+        else if (at >= 0) {
+            const int kv = hp / a.maps;
+            dst = (T*)a.k_pages + ((at + (long long)kv * a.page_size) * a.maps + (hp - kv * a.maps)) * a.dk;
+        }
+        if (j >= turning) {                              // dims that pass
+            const int d = a.rotary_dim + (j - turning) * VEC;
+            const uint4 raw = *reinterpret_cast<const uint4*>(src + d);
+            if (dst) *reinterpret_cast<uint4*>(dst + d) = raw;
+            continue;
+        }
+        const int d = j * VEC;
+        const uint4 lo = *reinterpret_cast<const uint4*>(src + d), hi = *reinterpret_cast<const uint4*>(src + half + d);
+        float x[VEC], y[VEC];
+        PrepVec<T>::widen(lo, x);
+        PrepVec<T>::widen(hi, y);
+        uint4 ra, rb;
+        T* pa = reinterpret_cast<T*>(&ra);
+        T* pb = reinterpret_cast<T*>(&rb);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float c = cs_sh[0][d + e], s = cs_sh[1][d + e];
+            pa[e] = lsb_from_float<T>(x[e] * c - y[e] * s);
+            pb[e] = lsb_from_float<T>(y[e] * c + x[e] * s);
+        }
+        if (dst) {
+            *reinterpret_cast<uint4*>(dst + d) = ra;
+            *reinterpret_cast<uint4*>(dst + half + d) = rb;
+        }
+    }
+}
+
 LSB_API int lsb_attention_prep_max_dim() { return kPrepMaxDim; }
 
 LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_off, int k_off, int v_off, int tokens,
@@ -289,6 +365,11 @@ LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_
     const int per16 = dtype == LSB_F32 ? 4 : 8;
     a.vec = ((uintptr_t)proj % 16 == 0 && (uintptr_t)v_pages % 16 == 0 && ld % per16 == 0 && q_off % per16 == 0 &&
              k_off % per16 == 0 && v_off % per16 == 0 && dk % per16 == 0 && dv % per16 == 0) ? 1 : 0;
+    if (a.vec && !q_bias && !k_bias && !v_bias && !q_norm && !k_norm && !v_unit && temp_every <= 0 && !v_first && !adjacent &&
+        (rotary_dim / 2) % per16 == 0 && (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0) {
+        LSB_DISPATCH_DTYPE(dtype, return lsb_launch(attention_prep_rotate_kernel<T>, dim3(tokens), dim3(kPrepWarps * 32), 0,
+                                                    stream, 1, a));
+    }
     const size_t smem = (size_t)(nh + nkv) * maps * dk * sizeof(float);
     if (smem > 160 * 1024) return (int)cudaErrorInvalidValue;
     LSB_DISPATCH_DTYPE(dtype, {

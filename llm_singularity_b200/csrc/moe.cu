@@ -58,9 +58,69 @@ struct RouteOpts {
 
 constexpr int kMaxTop = 32;
 
+// One warp chooses for one token, up to 128 experts: the logits in registers, four a lane, a chosen one struck
+// out; lane k keeps what the k-th choice was.
+__device__ __forceinline__ void route_token_small(const float* __restrict__ z, int E, int top, const RouteOpts& ro,
+                                                  int* __restrict__ ids, float* __restrict__ wts, int lane) {
+    float zv[4], cv[4], zmax = -FLT_MAX, denom = 1.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int e = lane + 32 * i;
+        zv[i] = -FLT_MAX;
+        if (e < E) zv[i] = ro.joins && ro.bias ? z[e] + ro.bias[e] : z[e];
+        zmax = fmaxf(zmax, zv[i]);
+    }
+    zmax = lsb_warp_max(zmax);
+    if (ro.score == 1) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s += lane + 32 * i < E ? expf(zv[i] - zmax) : 0.f;
+        denom = lsb_warp_sum(s);
+    }
+    auto score_of = [&](float v) {          // (score 2: relative to the largest logit, which is always chosen)
+        return ro.score == 0 ? 1.f / (1.f + expf(-v)) : expf(v - zmax) / denom;
+    };
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int e = lane + 32 * i;
+        cv[i] = e < E ? (ro.bias && !ro.joins ? score_of(zv[i]) + ro.bias[e] : zv[i]) : -FLT_MAX;
+    }
+    unsigned gone = 0;                      // bit i: this lane's i-th expert is chosen (or there is none)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+        if (lane + 32 * i >= E) gone |= 1u << i;
+    float mine = 0.f, total = 0.f;
+    int my_id = 0;
+    for (int k = 0; k < top; ++k) {
+        float best = -FLT_MAX, bz = 0.f;
+        int bi = 0x7fffffff;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (!(gone >> i & 1) && (bi == 0x7fffffff || cv[i] > best)) { best = cv[i]; bz = zv[i]; bi = lane + 32 * i; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o), oz = __shfl_xor_sync(0xffffffffu, bz, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (oi != 0x7fffffff && (bi == 0x7fffffff || ob > best || (ob == best && oi < bi))) { best = ob; bz = oz; bi = oi; }
+        }
+        if ((bi & 31) == lane) gone |= 1u << (bi >> 5);
+        const float v = score_of(bz);
+        if (lane == k) { mine = v; my_id = bi; }
+        total += v;
+    }
+    if (lane < top) {
+        ids[lane] = my_id;
+        wts[lane] = (ro.score == 2 ? mine / total : ro.renorm ? mine / (total + ro.eps) : mine) * ro.scale;
+    }
+}
+
 // One warp chooses for one token (all lanes call it together).
 __device__ __forceinline__ void route_token(const float* __restrict__ z, int E, int top, const RouteOpts ro,
                                             int* __restrict__ ids, float* __restrict__ wts, int lane) {
+    if (E <= 128) {
+        route_token_small(z, E, top, ro, ids, wts, lane);
+        return;
+    }
     const int score = ro.score, renorm = ro.renorm;
     const float* add = ro.joins ? ro.bias : nullptr;         // part of the logits
     const float* correct = ro.joins ? nullptr : ro.bias;     // for the choice alone
@@ -117,7 +177,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int n_tokens,
     route_token(logits + (size_t)warp * ro.ld, E, top, ro, ids + (size_t)warp * top, wts + (size_t)warp * top, lane);
 }
 
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(1024, 1)
 moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top, int E,
                  int cap_tiles, int tile, int* __restrict__ pos, int* __restrict__ row_token,
                  float* __restrict__ row_scale, int* __restrict__ tile_expert,
@@ -143,13 +203,21 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
         pos[i] = atomicAdd(&counts[e], 1);
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
+    if (threadIdx.x < 32) {                 // running sum over the experts, a warp's width at a time
+        const int lane = threadIdx.x;
         int at = 0;
-        for (int e = 0; e < E; ++e) {
-            starts[e] = at;
-            at += (counts[e] + tile - 1) / tile * tile;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int n_rows = e0 + lane < E ? (counts[e0 + lane] + tile - 1) / tile * tile : 0;
+            int sum = n_rows;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int below = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += below;
+            }
+            if (e0 + lane < E) starts[e0 + lane] = at + sum - n_rows;
+            at += __shfl_sync(0xffffffffu, sum, 31);
         }
-        starts[E] = at;
+        if (lane == 0) starts[E] = at;
     }
     __syncthreads();
     for (int e = threadIdx.x; e < E; e += blockDim.x)
@@ -282,6 +350,59 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
     }
 }
 
+// The same for bfloat16 rows of a multiple of 8 columns: 16 bytes a thread, a token's choices eight at a time with
+// all their rows in flight.
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ wts,
+                       int on_output, int top, int n, int capacity, __nv_bfloat16* __restrict__ out,
+                       const __nv_bfloat16* __restrict__ add, const float* __restrict__ add_gate, int gate_ld) {
+    lsb_pdl_launch_dependents();
+    lsb_pdl_wait();
+    const size_t t = blockIdx.x;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+    if (c >= n) return;
+    float s[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    auto join = [&](const uint4& raw, float w) {
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 f = __bfloat1622float2(p[j]);
+            s[2 * j] += w * f.x;
+            s[2 * j + 1] += w * f.y;
+        }
+    };
+    uint4 shared_row = make_uint4(0u, 0u, 0u, 0u);
+    float ag = 1.f;
+    if (add) {
+        shared_row = *reinterpret_cast<const uint4*>(add + t * n + c);
+        if (add_gate) ag = add_gate[t * gate_ld];
+    }
+    for (int k0 = 0; k0 < top; k0 += 8) {
+        uint4 rows[8];
+        float w[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            rows[k] = make_uint4(0u, 0u, 0u, 0u);
+            w[k] = 0.f;
+            if (k0 + k < top) {
+                const int p = pos[t * top + k0 + k];
+                if (p >= 0 && p < capacity) {
+                    rows[k] = *reinterpret_cast<const uint4*>(y + (size_t)p * n + c);
+                    w[k] = on_output ? wts[t * top + k0 + k] : 1.f;
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            if (k0 + k < top) join(rows[k], w[k]);
+    }
+    if (add) join(shared_row, add_gate ? 1.f / (1.f + expf(-ag)) : 1.f);
+    __nv_bfloat162 o[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] = __floats2bfloat162_rn(s[2 * j], s[2 * j + 1]);
+    *reinterpret_cast<uint4*>(out + t * n + c) = *reinterpret_cast<const uint4*>(o);
+}
+
 LSB_API int lsb_moe_tile() { return kTile; }
 
 LSB_API int lsb_moe_route(const float* logits, int ld, int n_tokens, int E, int top, int score, int renorm,
@@ -353,6 +474,13 @@ LSB_API int lsb_moe_combine(const void* y, int y_same, const int* pos, const flo
                             int n_tokens, int top, int n, int capacity, void* out, int dtype, const void* add,
                             const float* add_gate, int gate_ld, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (dtype == LSB_BF16 && y_same && n % 8 == 0 &&
+        (((uintptr_t)y | (uintptr_t)out | (uintptr_t)add) & 15) == 0) {
+        const int chunks = n / 8, threads = chunks >= 256 ? 256 : (chunks + 31) / 32 * 32;
+        return lsb_launch(moe_combine_vec_kernel, dim3(n_tokens, (chunks + threads - 1) / threads), dim3(threads), 0, stream, 1,
+                          (const __nv_bfloat16*)y, pos, wts, on_output, top, n, capacity, (__nv_bfloat16*)out,
+                          (const __nv_bfloat16*)add, add_gate, gate_ld);
+    }
     LSB_DISPATCH_DTYPE(dtype, {
         if (y_same)
             return lsb_launch(moe_combine_kernel<T, T>, dim3(n_tokens), dim3(256), 0, stream, 1, (const T*)y, pos,

@@ -702,30 +702,40 @@ def _fork_join(ctx, device):
     return got
 
 
-OVERLAP_SUBLAYERS = 64          # steps of at most this many tokens run independent sublayers on two streams (0: none)
-_branch: Dict[torch.device, tuple] = {}
+OVERLAP_SUBLAYERS = 64          # steps of at most this many tokens run independent sublayers on streams of their own (0: none)
+_branches: Dict[torch.device, list] = {}      # free (stream, event, event) triples
+
+
+def fork(rows: int, device, fn):
+    """Start ``fn()``, a chain of kernels that does not depend on what the caller launches next; returns ``join``,
+    which gives its result once the caller's stream is behind it.  In a step of few rows, whose kernels wait
+    on memory and on one another, the chain runs on a stream of its own; in others ``join`` runs it.  What
+    the chain allocates lives on its stream and what it reads must be kept until ``join``, so that memory
+    handed back is only ever reused behind its last use."""
+    if _recording is not None or not 0 < rows <= OVERLAP_SUBLAYERS:
+        return fn
+    free = _branches.setdefault(device, [])
+    side, began, done = branch = free.pop() if free else (torch.cuda.Stream(device), torch.cuda.Event(), torch.cuda.Event())
+    here = torch.cuda.current_stream(device)
+    began.record(here)
+    side.wait_event(began)
+    with torch.cuda.stream(side):
+        result = fn()
+        done.record(side)
+
+    def join():
+        here.wait_event(done)
+        free.append(branch)
+        return result
+
+    return join
 
 
 def side_by_side(rows: int, device, first, second):
-    """(first(), second()), two chains of kernels that do not depend on one another: in a step of few rows, whose
-    kernels wait on memory and on one another, the second runs on a stream of its own beside the first.
-    What either allocates is used on its own stream until both have joined again, so that memory handed
-    back is only ever reused behind its last use."""
-    if _recording is not None or not 0 < rows <= OVERLAP_SUBLAYERS:
-        return first(), second()
-    got = _branch.get(device)
-    if got is None:
-        got = _branch[device] = (torch.cuda.Stream(device), torch.cuda.Event(), torch.cuda.Event())
-    side, fork, join = got
-    here = torch.cuda.current_stream(device)
-    fork.record(here)
-    side.wait_event(fork)
-    with torch.cuda.stream(side):
-        b = second()
-        join.record(side)
+    """(first(), second()) of two chains of kernels that do not depend on one another, the second as a fork."""
+    join = fork(rows, device, second)
     a = first()
-    here.wait_event(join)
-    return a, b
+    return a, join()
 
 
 def _batch_shape(ctx):
@@ -1931,6 +1941,10 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     y = torch.empty(cap_tiles * tile, H, dtype=x.dtype if tc else torch.float32, device=dev)
     s = _stream(out)
     on_input = 1 if weight_on == "input" else 0
+    # a shared expert's rows: on a stream of their own in a step of few tokens, else made behind the experts'
+    # products (its own products' weights are then the last streamed before the next layer's, which they ask
+    # L2 for while they end)
+    add_join = fork(T, dev, add) if callable(add) else None
     r_logits, r_score, r_renorm, r_bias, r_scale, r_eps, r_joins = (tuple(route) + (None, 1.0, 0.0, False)[len(route) - 3:])[:7] \
         if route is not None else (None, 0, 0, None, 1.0, 0.0, False)
     if r_logits is not None and (r_logits.shape[0] != T or r_logits.shape[1] < E):
@@ -1952,8 +1966,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
               _p(tile_expert), _i(cap_tiles), _p(hidden), _i(F), _i(H), _i(act), _f(limit), _i(0 if gated else 1), s)
         _call("moe", "lsb_moe_down", _p(hidden), _i(_dt(x)), _p(row_token), _p(w_down), _p(tile_expert), _i(cap_tiles),
               _p(y), _i(H), _i(F), s)
-    if callable(add):           # made now, behind the experts' products (its own products' weights are then the
-        add = add()             # last streamed before the next layer's, which they ask L2 for while they end)
+    if add_join is not None:
+        add = add_join()
     if add is not None:
         _req(add, "add", x.dtype, 2)
         if add.shape != (T, H):
