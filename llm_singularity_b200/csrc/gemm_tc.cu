@@ -208,8 +208,17 @@ __device__ __forceinline__ float plain_act(float z, int act) {
     return __fdividef(z, 1.f + __expf(-a));
 }
 __device__ __forceinline__ void plain_act_all(uint32_t (&r)[32], int act) {
+    // (the choice outside the loop: inside, every value would carry it)
+    if (act == LSB_ACT_RELU_SQUARED) {
 #pragma unroll
-    for (int x = 0; x < 32; ++x) r[x] = __float_as_uint(plain_act(__uint_as_float(r[x]), act));
+        for (int x = 0; x < 32; ++x) r[x] = __float_as_uint(plain_act(__uint_as_float(r[x]), LSB_ACT_RELU_SQUARED));
+    } else if (act == LSB_ACT_GELU_TANH) {
+#pragma unroll
+        for (int x = 0; x < 32; ++x) r[x] = __float_as_uint(plain_act(__uint_as_float(r[x]), LSB_ACT_GELU_TANH));
+    } else {
+#pragma unroll
+        for (int x = 0; x < 32; ++x) r[x] = __float_as_uint(plain_act(__uint_as_float(r[x]), LSB_ACT_SILU));
+    }
 }
 #define silu_mul(g, u) gate_mul((g), (u), prm.act, prm.limit)
 

@@ -224,6 +224,28 @@ def test_greedy_generation_through_the_engine(tmp_path, dtype, name="mix_a"):
     assert clear > new
 
 
+def test_requests_share_the_pages_of_a_common_prefix(tmp_path, name="mix_b"):
+    """Every cache of the design is full pages, a looped layer's passes included, so a second request with the
+    same first tokens takes them from the prefix tree and generates what the plain model picks."""
+    from llm_singularity_b200 import Engine
+    cfg = U.CONFIGS[name]
+    W, path = _setup(tmp_path, cfg, 37)
+    eng = Engine(path, dtype="float32", kv_block_size=16, num_kv_blocks=32, max_batch_size=2, max_tokens_per_batch=64)
+    assert eng.prefix is not None
+    common = U.tokens_for(cfg, 40, 3)
+    for k, tail in enumerate(([5, 9, 2], [7, 1])):
+        rid = eng.add_request(common + tail, max_new_tokens=5)
+        seq = common + tail
+        while eng.has_work():
+            for r, tok, _ in eng.step():
+                assert r == rid
+                top2 = torch.topk(U.plain_logits(cfg, W, seq)[-1], 2)
+                if top2.values[0] - top2.values[1] > 0.05:
+                    assert tok == int(top2.indices[0]), (k, len(seq))
+                seq.append(tok)
+        assert eng.prefix.hits == 2 * k
+
+
 # ----------------------------------------------------------------- kernels against plain functions
 def _ctx(q_lens, kv_lens, rows=None):
     from llm_singularity_b200.engine.batch import ContextBuilder
