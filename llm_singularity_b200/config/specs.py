@@ -113,9 +113,11 @@ class LinearRecurrenceSpec(PartSpec):
     and b is a key projection; "forget": a is a forget gate per channel with a learnt floor,
     ``a = floor + (1 - floor) * sigmoid(W_f x + bias)``, and ``b = 1 - a`` (no key).  The
     activations of the query, key and value projections, how the output is normed (over all heads
-    together, "all", or each head by itself with one weight of head size, "per_head") and whether a
-    sigmoid gate projection multiplies it are fields, so that relatives of the two shipped kinds
-    (``lightning`` and ``hgrn2``) are other settings of the same part."""
+    together, "all", each head by itself with one weight of head size, "per_head", or each head by
+    itself without a weight, "unit") and whether a gate projection multiplies it, through
+    ``out_gate_activation`` ("sigmoid" or "silu"), are fields, so that relatives of the shipped kinds
+    (``lightning``, ``hgrn2`` and retention) are other settings of the same part.  ``position``: a rotation
+    of every head of q and k (a fixed decay only); ``k_scale`` multiplies k."""
 
     hidden_size: int = 0
     num_heads: int = 0
@@ -129,7 +131,34 @@ class LinearRecurrenceSpec(PartSpec):
     out_norm: str = "all"
     out_gate: bool = False
     eps: float = 1e-5
+    out_gate_activation: str = "sigmoid"
+    position: PartSpec = field(default_factory=NoPositionSpec)
+    k_scale: float = 1.0
     kind: str = field(init=False, default="linear_recurrence")
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec(PartSpec):
+    """A state-space memory with one fade per head and token (the Mamba-2 cell).  One projection makes
+    ``[z | x | B | C | dt]``: z and x of ``num_heads * value_dim``, B and C of ``groups * state_dim`` (head h
+    reads group ``h // (num_heads / groups)``), dt one number per head.  x, B and C together pass a causal
+    convolution over time per channel (``conv_taps`` taps, a bias, zeros before the start) and silu; with
+    ``dt <- softplus(dt + dt_bias)``
+
+        S <- exp(-exp(A_log) dt) S + dt B x^T;   y = S^T C + D x
+
+    y times silu(z) is RMS-normed in ``norm_groups`` equal parts (``eps``) with one weight over all heads,
+    then projected by W_o."""
+
+    hidden_size: int = 0
+    num_heads: int = 0
+    groups: int = 1
+    state_dim: int = 0
+    value_dim: int = 0            # per head
+    conv_taps: int = 1
+    norm_groups: int = 1
+    eps: float = 1e-5
+    kind: str = field(init=False, default="state_space")
 
 
 @dataclass(frozen=True)
@@ -157,7 +186,10 @@ class KVAttentionSpec(PartSpec):
     side, [map 1, map 2]) over one value; with a_m the attention of map m, the head's output is
     ``unit(a_1 - lambda a_2) * (1 - diff)``, ``unit`` the division by the root mean square over the
     head (``eps``), and ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` one number of the layer
-    made of four learnt vectors of ``key_dim``.  It goes with position, window and chunk only."""
+    made of four learnt vectors of ``key_dim``.  It goes with position, window and chunk only.
+    ``qk_unit``: every head of q and k is divided by its root mean square (``eps``, no weight); a rotation
+    keeps the length, so before or after it is the same.  ``sink_logit``: the sink's score is a learnt
+    number per head instead of 0 (it is not scaled).  ``out_bias``: the output projection has a bias."""
 
     hidden_size: int = 0
     num_heads: int = 0
@@ -183,6 +215,9 @@ class KVAttentionSpec(PartSpec):
     sink: bool = False
     gate_per_head: bool = False
     diff: Optional[float] = None
+    qk_unit: bool = False
+    sink_logit: bool = False
+    out_bias: bool = False
     kind: str = field(init=False, default="kv_attention")
 
 
@@ -355,7 +390,8 @@ class MoESpec(PartSpec):
     ``renorm_eps`` and multiplied by ``weight_scale``.  ``limit`` belongs to the activation
     "capped_glu" (see ``GatedMLPSpec``).  ``shared``: a feed-forward that every token passes
     besides its chosen experts; its result is added, multiplied by sigmoid(W_sg x), one number per token,
-    with ``shared_gate``."""
+    with ``shared_gate``.  ``token_rows`` R > 0: no router; a table of integers [R, ``top``] names the experts
+    of every token id (R is the vocabulary's size), each with the weight ``1 / top``."""
 
     hidden_size: int = 0
     expert_size: int = 0
@@ -373,6 +409,7 @@ class MoESpec(PartSpec):
     gated: bool = True
     router_bias: bool = False
     shared_gate: bool = False
+    token_rows: int = 0
     kind: str = field(init=False, default="moe")
 
 
@@ -446,6 +483,18 @@ class SandwichBlockSpec(PartSpec):
     ffn_post_norm: Optional[PartSpec] = None
     residual_mult: float = 1.0
     kind: str = field(init=False, default="sandwich_norm")
+
+
+@dataclass(frozen=True)
+class OutputNormBlockSpec(PartSpec):
+    """x += norm1(mixer(x)); x += norm2(ffn(x))   (the "output_norm" arrangement: the sublayers read the
+    stream itself, a norm stands behind each).  ``ffn`` None: no second step."""
+
+    mixer: PartSpec = None
+    ffn: Optional[PartSpec] = None
+    mixer_norm: PartSpec = None
+    ffn_norm: Optional[PartSpec] = None
+    kind: str = field(init=False, default="output_norm")
 
 
 @dataclass(frozen=True)

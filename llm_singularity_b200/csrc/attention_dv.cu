@@ -12,7 +12,8 @@
 // kDvLinearBias takes slope_h * (p - j) off the score of key j for the query at p, slope_h = 2^(-8 (h + 1) / nh);
 // `softcap` > 0 replaces a scaled score s by softcap * tanh(s / softcap) before that.
 // kDvSink adds one to the softmax's denominator (a place with score 0 and no value, so a row's weights
-// sum to less than one), kDvGateHeads reads one gate number per head, gate[t, h], instead of one per
+// sum to less than one), or exp(sink_logit[h]) where such scores are given (32-bit, one per query head, not
+// scaled), kDvGateHeads reads one gate number per head, gate[t, h], instead of one per
 // output channel.
 //
 // Generic form (any sizes, 32-bit or bfloat16 storage): one warp owns a (row, head); lanes split
@@ -45,7 +46,7 @@ attention_dv_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pag
                             const int* __restrict__ table_rows, const int* __restrict__ block_table, int table_stride,
                             const T* __restrict__ gate, long long gate_stride, T* __restrict__ out,
                             int nh, int nkv, int dk, int dv, int page_size, int num_pages, float scale, int window,
-                            int chunk, int vec, int flags, float softcap) {
+                            int chunk, int vec, int flags, float softcap, const float* __restrict__ sink_logit) {
     __shared__ float q_sh[kDvWarps][kDvMaxDim];
     lsb_pdl_launch_dependents();
     lsb_pdl_wait();
@@ -109,7 +110,7 @@ attention_dv_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pag
         }
         m = m_new;
     }
-    if (flags & kDvSink) l += expf(-m);                      // the sink's weight relative to the maximum (inf: all weights vanish)
+    if (flags & kDvSink) l += expf((sink_logit ? sink_logit[h] : 0.f) - m);     // the sink's weight relative to the maximum (inf: all weights vanish)
     const float inv = l > 0.f ? 1.f / l : 0.f;
     T* o = out + ((size_t)t * nh + h) * dv;
     const bool per_head = (flags & kDvGateHeads) != 0;
@@ -137,7 +138,7 @@ attention_dv_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                         const __nv_bfloat16* __restrict__ gate, long long gate_stride,
                         __nv_bfloat16* __restrict__ out, int nh, int nkv, int dk, int dv, int page_size,
                         int num_pages, float scale_log2, int window, int chunk, int ksplit, float* __restrict__ scratch,
-                        int flags, float scale, float softcap) {
+                        int flags, float scale, float softcap, const float* __restrict__ sink_logit) {
     constexpr int KS = DKP + 8, VS = DVP + 8;          // row strides in elements: 4 words past a multiple of 32
     extern __shared__ __align__(16) unsigned char dv_smem[];
     __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(dv_smem);       // [STAGES][64][KS]
@@ -425,10 +426,10 @@ attention_dv_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                 }
                 continue;
             }
-            if (sink) den += exp2f(-mm);
-            float y = den > 0.f ? num / den : 0.f;
             const size_t t = (size_t)qs + row / group;
             const int h = g * group + row % group;
+            if (sink) den += exp2f((sink_logit ? sink_logit[h] * 1.4426950408889634f : 0.f) - mm);
+            float y = den > 0.f ? num / den : 0.f;
             if (gate) y *= 1.f / (1.f + __expf(-__bfloat162float(gate[t * gate_stride + (size_t)h * gate_w + (per_head ? 0 : c)])));
             out[(t * nh + h) * dv + c] = __float2bfloat16_rn(y);
         }
@@ -436,8 +437,8 @@ attention_dv_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     }
     if (!active) return;
     if (sink) {
-        l_a += exp2f(-m_a);
-        l_b += exp2f(-m_b);
+        l_a += exp2f((sink_logit ? sink_logit[h_a] * 1.4426950408889634f : 0.f) - m_a);
+        l_b += exp2f((sink_logit ? sink_logit[h_b] * 1.4426950408889634f : 0.f) - m_b);
     }
     const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
     float gh_a = 1.f, gh_b = 1.f;                      // one gate number per head
@@ -476,7 +477,8 @@ attention_dv_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
 __global__ void __launch_bounds__(kMmaThreads)
 attention_dv_merge_kernel(const float* __restrict__ scratch, const int* __restrict__ q_start,
                           const __nv_bfloat16* __restrict__ gate, long long gate_stride,
-                          __nv_bfloat16* __restrict__ out, int nh, int nkv, int dv, int ksplit, int flags) {
+                          __nv_bfloat16* __restrict__ out, int nh, int nkv, int dv, int ksplit, int flags,
+                          const float* __restrict__ sink_logit) {
     lsb_pdl_launch_dependents();
     lsb_pdl_wait();
     const int r = blockIdx.z, g = blockIdx.y, group = nh / nkv;
@@ -507,10 +509,10 @@ attention_dv_merge_kernel(const float* __restrict__ scratch, const int* __restri
             num += f * pv[p];
             den += f * pl[p];
         }
-        if (flags & kDvSink) den += exp2f(-mm);
-        float y = den > 0.f ? num / den : 0.f;
         const size_t t = (size_t)qs + row / group;
         const int h = g * group + row % group;
+        if (flags & kDvSink) den += exp2f((sink_logit ? sink_logit[h] * 1.4426950408889634f : 0.f) - mm);
+        float y = den > 0.f ? num / den : 0.f;
         const bool per_head = (flags & kDvGateHeads) != 0;
         if (gate) y *= 1.f / (1.f + __expf(-__bfloat162float(gate[t * gate_stride + (per_head ? (size_t)h : (size_t)h * dv + c)])));
         out[(t * nh + h) * dv + c] = __float2bfloat16_rn(y);
@@ -532,7 +534,7 @@ LSB_API int lsb_attention_dv_mma(const void* q, const void* k_pages, const void*
                                  const void* gate, long long gate_stride, void* out, int n_requests, int max_q_len,
                                  int nh, int nkv, int dk, int dv, int page_size, int num_pages, float scale, int window,
                                  int chunk, int sms, int shape, float* scratch, int flags, float softcap,
-                                 cudaStream_t stream) {
+                                 const float* sink_logit, cudaStream_t stream) {
     if (n_requests <= 0 || max_q_len <= 0) return 0;
     if (sms <= 0) sms = 148;
     if (!lsb_attention_dv_mma_supported(dk, dv) || nkv <= 0 || nh % nkv || window < 0 || chunk < 0 || n_requests > 65535 ||
@@ -559,7 +561,7 @@ LSB_API int lsb_attention_dv_mma(const void* q, const void* k_pages, const void*
                           stream, 1, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,                     \
                           (const __nv_bfloat16*)v_pages, q_start, kv_len, table_rows, block_table, table_stride, \
                           (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, nh, nkv, dk, dv,         \
-                          page_size, num_pages, scale_log2, window, chunk, ksplit, scratch, flags, scale, softcap);              \
+                          page_size, num_pages, scale_log2, window, chunk, ksplit, scratch, flags, scale, softcap, sink_logit);  \
     } while (0)
 #define LSB_DV_MMA_SHAPE(DKP, DVP)                                                                               \
     do {                                                                                                         \
@@ -582,7 +584,7 @@ LSB_API int lsb_attention_dv_mma(const void* q, const void* k_pages, const void*
     if (rc || ksplit <= 1) return rc;
     return lsb_launch(attention_dv_merge_kernel, dim3(tiles, nkv, n_requests), dim3(kMmaThreads), 0, stream, 1,
                       (const float*)scratch, q_start, (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)out, nh, nkv,
-                      dv, ksplit, flags);
+                      dv, ksplit, flags, sink_logit);
 }
 
 LSB_API int lsb_attention_dv_max_dim() { return kDvMaxDim; }
@@ -594,7 +596,7 @@ LSB_API int lsb_attention_dv_generic(const void* q, const void* k_pages, const v
                                      int table_stride, const void* gate, long long gate_stride, void* out, int dtype,
                                      int n_requests, int max_q_len, int nh, int nkv, int dk, int dv, int page_size,
                                      int num_pages, float scale, int window, int chunk, int flags, float softcap,
-                                     cudaStream_t stream) {
+                                     const float* sink_logit, cudaStream_t stream) {
     if (n_requests <= 0 || max_q_len <= 0) return 0;
     if (dk <= 0 || dk > kDvMaxDim || dv <= 0 || dv > kDvMaxDim || nkv <= 0 || nh % nkv || window < 0 || chunk < 0)
         return (int)cudaErrorInvalidValue;
@@ -605,6 +607,6 @@ LSB_API int lsb_attention_dv_generic(const void* q, const void* k_pages, const v
     LSB_DISPATCH_DTYPE(dtype, return lsb_launch(
         attention_dv_generic_kernel<T>, grid, dim3(kDvWarps * 32), 0, stream, 1, (const T*)q, (const T*)k_pages,
         (const T*)v_pages, q_start, kv_len, table_rows, block_table, table_stride, (const T*)gate, gate_stride,
-        (T*)out, nh, nkv, dk, dv, page_size, num_pages, scale, window, chunk, vec, flags, softcap));
+        (T*)out, nh, nkv, dk, dv, page_size, num_pages, scale, window, chunk, vec, flags, softcap, sink_logit));
     return 0;
 }

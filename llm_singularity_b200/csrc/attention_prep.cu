@@ -4,7 +4,8 @@
 //   * a bias per channel (q, k, v), added in 32-bit;
 //   * a norm per head of q and of k: z / sqrt(mean(z^2) + eps) * w, one weight of head size for
 //     all heads of q and one for all heads of k; or (`norm_all`) one norm over all heads of q at
-//     once and one over all heads of k, with weights as long as the whole projection;
+//     once and one over all heads of k, with weights as long as the whole projection; or (`qk_unit`) the norm
+//     per head without a weight;
 //   * each value head divided by its root mean square (`v_unit`: no weight, the same eps);
 //   * values mixed with those another layer made of the same token in this step (`v_first`, rows of
 //     `v_first_ld` elements in the compute dtype): v <- (1 - lambda) v + lambda v_first, lambda one
@@ -35,7 +36,7 @@ struct PrepArgs {
     int nh, nkv, dk, dv, maps;
     const float *q_bias, *k_bias, *v_bias;
     const float *q_norm, *k_norm; float norm_eps;
-    int norm_all, v_unit;
+    int norm_all, v_unit, qk_unit;
     float temp_coef; int temp_every;
     const float* inv_freq; int rotary_dim, adjacent;
     const int *positions, *token_req, *table_rows, *block_table; int table_stride;
@@ -179,7 +180,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
         float inv = 1.f;
         if (nw && a.norm_all) {
             inv = is_q ? inv_all_q : inv_all_k;
-        } else if (nw) {
+        } else if (nw || a.qk_unit) {
             float ss = 0.f;
             for (int d = lane; d < a.dk; d += 32) ss += hs[d] * hs[d];
             inv = rsqrtf(lsb_warp_sum(ss) / (float)a.dk + a.norm_eps);
@@ -203,8 +204,8 @@ __global__ void __launch_bounds__(kPrepWarps * 32) attention_prep_kernel(PrepArg
                     ia = a.rotary_dim + 2 * (i - half_rot);
                     ib = ia + 1;
                 }
-                float x0 = hs[ia] * (nw ? inv * nw[ia] : 1.f) * mul;
-                float x1 = ib < a.dk ? hs[ib] * (nw ? inv * nw[ib] : 1.f) * mul : 0.f;
+                float x0 = hs[ia] * (nw ? inv * nw[ia] : inv) * mul;
+                float x1 = ib < a.dk ? hs[ib] * (nw ? inv * nw[ib] : inv) * mul : 0.f;
                 if (i < half_rot) {
                     const float c = cs_sh[0][i], s = cs_sh[1][i];
                     const float r0 = x0 * c - x1 * s, r1 = x1 * c + x0 * s;
@@ -340,21 +341,21 @@ LSB_API int lsb_attention_prep_max_dim() { return kPrepMaxDim; }
 LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_off, int k_off, int v_off, int tokens,
                                int nh, int nkv, int dk, int dv, const float* q_bias, const float* k_bias,
                                const float* v_bias, const float* q_norm, const float* k_norm, float norm_eps,
-                               int norm_all, int v_unit, int maps, float temp_coef, int temp_every, const float* inv_freq, int rotary_dim, int adjacent,
+                               int norm_all, int v_unit, int qk_unit, int maps, float temp_coef, int temp_every, const float* inv_freq, int rotary_dim, int adjacent,
                                const int* positions, const int* token_req, const int* table_rows,
                                const int* block_table, int table_stride, void* q_out, void* k_pages, void* v_pages,
                                int page_size, int num_pages, int store, const void* v_first, long long v_first_ld,
                                const float* v_lambda, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (dk <= 0 || dk > kPrepMaxDim || maps < 1 || dv <= 0 || nh <= 0 || nkv <= 0 || rotary_dim % 2 || rotary_dim > dk ||
-        rotary_dim < 0 || (rotary_dim > 0 && !inv_freq) || (v_first && (!v_lambda || v_unit)))
+        rotary_dim < 0 || (rotary_dim > 0 && !inv_freq) || (v_first && (!v_lambda || v_unit)) || (qk_unit && (q_norm || k_norm)))
         return (int)cudaErrorInvalidValue;
     PrepArgs a;
     a.proj = proj; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
     a.nh = nh; a.nkv = nkv; a.dk = dk; a.dv = dv; a.maps = maps;
     a.q_bias = q_bias; a.k_bias = k_bias; a.v_bias = v_bias;
     a.q_norm = q_norm; a.k_norm = k_norm; a.norm_eps = norm_eps;
-    a.norm_all = norm_all; a.v_unit = v_unit;
+    a.norm_all = norm_all; a.v_unit = v_unit; a.qk_unit = qk_unit;
     a.temp_coef = temp_coef; a.temp_every = temp_every;
     a.inv_freq = inv_freq; a.rotary_dim = rotary_dim; a.adjacent = adjacent;
     a.positions = positions; a.token_req = token_req; a.table_rows = table_rows; a.block_table = block_table;
@@ -365,7 +366,7 @@ LSB_API int lsb_attention_prep(const void* proj, int dtype, long long ld, int q_
     const int per16 = dtype == LSB_F32 ? 4 : 8;
     a.vec = ((uintptr_t)proj % 16 == 0 && (uintptr_t)v_pages % 16 == 0 && ld % per16 == 0 && q_off % per16 == 0 &&
              k_off % per16 == 0 && v_off % per16 == 0 && dk % per16 == 0 && dv % per16 == 0) ? 1 : 0;
-    if (a.vec && !q_bias && !k_bias && !v_bias && !q_norm && !k_norm && !v_unit && temp_every <= 0 && !v_first && !adjacent &&
+    if (a.vec && !q_bias && !k_bias && !v_bias && !q_norm && !k_norm && !v_unit && !qk_unit && temp_every <= 0 && !v_first && !adjacent &&
         (rotary_dim / 2) % per16 == 0 && (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0) {
         LSB_DISPATCH_DTYPE(dtype, return lsb_launch(attention_prep_rotate_kernel<T>, dim3(tokens), dim3(kPrepWarps * 32), 0,
                                                     stream, 1, a));

@@ -44,6 +44,7 @@ struct AttnParams {
     int window;
     int skip_single;              // requests with one new token are left to the decode kernel
     int sink;                     // one more place with score 0 and no value in every softmax
+    const float* sink_logit;      // ... or with this score, one number a head, not scaled (or null)
     const bf16* gate;             // [tokens, heads] with this row stride: out *= sigmoid(gate), one number a head (or null)
     long long gate_stride;
     float softcap;                // > 0: a scaled score s becomes softcap * tanh(s / softcap)
@@ -420,7 +421,8 @@ prefill_attention_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __
         }
         if (ok) {
             // (the sink's share is 2^(0 - reference), the weight a key with score 0 would have had)
-            if (prm.sink) l += (m == -INFINITY) ? 1.f : exp2f(-m);
+            // (or one of the head's own sink score)
+            if (prm.sink) l += (m == -INFINITY) ? 1.f : exp2f((prm.sink_logit ? prm.sink_logit[h] * kLog2e : 0.f) - m);
             float inv = l > 0.f ? 1.f / l : 0.f;
             if (prm.gate != nullptr && live) {
                 const float z = __bfloat162float(prm.gate[(size_t)(qs + i0 + il) * prm.gate_stride + h]);
@@ -488,7 +490,7 @@ LSB_API int lsb_prefill_attention_tc5_biased(const void* qkv, int qkv_stride, in
                                              int n_requests, int max_q_len, int nh, int nkv, int hd, int page_size,
                                              int num_pages, float scale, int window, int skip_single, int sink,
                                              const void* gate, long long gate_stride, float softcap, int linear_bias,
-                                             cudaStream_t stream) {
+                                             const float* sink_logit, cudaStream_t stream) {
     if (n_requests <= 0 || max_q_len <= 0) return 0;
     if (!lsb_prefill_attention_tc5_supported(qkv, qkv_stride, k_pages, v_pages, nh, nkv, hd, page_size) ||
         n_requests > 65535 || (max_q_len + kRows - 1) / kRows > 65535)
@@ -513,7 +515,7 @@ LSB_API int lsb_prefill_attention_tc5_biased(const void* qkv, int qkv_stride, in
     prm.q_start = q_start; prm.kv_len = kv_len; prm.table_rows = table_rows; prm.block_table = block_table;
     prm.table_stride = table_stride; prm.out = (bf16*)out; prm.nh = nh; prm.nkv = nkv;
     prm.page_size = page_size; prm.num_pages = num_pages; prm.scale = scale; prm.window = window; prm.skip_single = skip_single;
-    prm.sink = sink; prm.gate = (const bf16*)gate; prm.gate_stride = gate_stride;
+    prm.sink = sink; prm.sink_logit = sink_logit; prm.gate = (const bf16*)gate; prm.gate_stride = gate_stride;
     prm.softcap = softcap; prm.linear_bias = linear_bias;
     int sh = 0;
     while ((1 << sh) < page_size) ++sh;
@@ -530,5 +532,5 @@ LSB_API int lsb_prefill_attention_tc5(const void* qkv, int qkv_stride, int n_tok
                                       const void* gate, long long gate_stride, cudaStream_t stream) {
     return lsb_prefill_attention_tc5_biased(qkv, qkv_stride, n_tokens, k_pages, v_pages, q_start, kv_len, table_rows,
                                             block_table, table_stride, out, n_requests, max_q_len, nh, nkv, hd, page_size,
-                                            num_pages, scale, window, skip_single, sink, gate, gate_stride, 0.f, 0, stream);
+                                            num_pages, scale, window, skip_single, sink, gate, gate_stride, 0.f, 0, nullptr, stream);
 }

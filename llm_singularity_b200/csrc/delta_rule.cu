@@ -480,9 +480,9 @@ delta_chain_kernel(float* __restrict__ state, int n_slots, const float* __restri
 // ------------------------------------------------------------------ read-out norm and gate
 // out[t, h, c] = x[t, h, c] / sqrt(mean_c x^2 + eps) * w[(h V + c) mod w_len] * act(gate[t, h V + c]);
 // gate_act 0: no gate, 1: sigmoid, 2: silu.  A warp per (token, head).
-template <typename T>
+template <typename T, typename TG>
 __global__ void __launch_bounds__(kDeltaThreads)
-delta_output_kernel(const float* __restrict__ x, const float* __restrict__ w, int w_len, const T* __restrict__ gate,
+delta_output_kernel(const float* __restrict__ x, const float* __restrict__ w, int w_len, const TG* __restrict__ gate,
                     long long gate_stride, int gate_act, T* __restrict__ out, long long pairs, int H, int V, float eps) {
     lsb_pdl_launch_dependents();
     lsb_pdl_wait();
@@ -496,7 +496,7 @@ delta_output_kernel(const float* __restrict__ x, const float* __restrict__ w, in
     for (int c = lane; c < V; c += 32) ss += xr[c] * xr[c];
     const float inv = rsqrtf(lsb_warp_sum(ss) / (float)V + eps);
     for (int c = lane; c < V; c += 32) {
-        float y = xr[c] * inv * w[(h * V + c) % w_len];
+        float y = xr[c] * inv * (w ? w[(h * V + c) % w_len] : 1.f);
         if (gate_act) {
             const float z = lsb_to_float(gate[t * gate_stride + (long long)h * V + c]);
             y *= gate_act == 1 ? delta_sigmoid(z) : z * delta_sigmoid(z);
@@ -644,15 +644,21 @@ LSB_API int lsb_delta_scan(int mode, const float* vecs, const float* scal, const
     return 0;
 }
 
+// w may be null (no weight); gate_f32: the gate's rows are 32-bit whatever out's type is
 LSB_API int lsb_delta_output(const float* x, const float* w, int w_len, const void* gate, long long gate_stride,
-                             int gate_act, void* out, int dtype, int tokens, int H, int V, float eps, cudaStream_t stream) {
+                             int gate_act, int gate_f32, void* out, int dtype, int tokens, int H, int V, float eps, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (H <= 0 || V <= 0 || w_len <= 0 || gate_act < 0 || gate_act > 2 || (gate_act && !gate)) return (int)cudaErrorInvalidValue;
     const long long pairs = (long long)tokens * H;
     const long long blocks = (pairs + kDeltaThreads / 32 - 1) / (kDeltaThreads / 32);
     if (blocks > 0x7fffffffLL) return (int)cudaErrorInvalidValue;
-    LSB_DISPATCH_DTYPE(dtype, return lsb_launch(delta_output_kernel<T>, dim3((unsigned)blocks), dim3(kDeltaThreads), 0, stream, 1,
-                                                x, w, w_len, (const T*)gate, gate_stride, gate_act, (T*)out, pairs, H, V, eps));
+    LSB_DISPATCH_DTYPE(dtype, {
+        if (gate_f32)
+            return lsb_launch(delta_output_kernel<T, float>, dim3((unsigned)blocks), dim3(kDeltaThreads), 0, stream, 1, x, w, w_len,
+                              (const float*)gate, gate_stride, gate_act, (T*)out, pairs, H, V, eps);
+        return lsb_launch(delta_output_kernel<T, T>, dim3((unsigned)blocks), dim3(kDeltaThreads), 0, stream, 1, x, w, w_len,
+                          (const T*)gate, gate_stride, gate_act, (T*)out, pairs, H, V, eps);
+    });
     return 0;
 }
 

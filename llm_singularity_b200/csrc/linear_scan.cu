@@ -16,6 +16,8 @@
 //                          has V + 1 columns and the last column of the output is (sum of b) . q
 //   q = act_q(q projection) * q_scale, v = act_v(v projection); act: 0 none, 1 silu
 //
+// q and k may be shared by the heads of a group: head h reads q and k head h / (heads / key_heads).
+//
 // A block owns (request, head, a tile of value columns) and walks the request's tokens in order,
 // so the result does not depend on how a prompt was cut into steps.  A column's key channels are
 // dealt to `split` neighbouring lanes (channel d = lane_part * per_thread + i), each keeping its
@@ -87,7 +89,8 @@ linear_scan_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
                    const int* __restrict__ q_start, const int* __restrict__ table_rows,
                    float* __restrict__ out, int split, int vec, int seg_len, int max_segs,
                    float* __restrict__ seg_state, float* __restrict__ seg_decay,
-                   const float* __restrict__ g_keep, const float* __restrict__ g_write, int ones, float q_scale) {
+                   const float* __restrict__ g_keep, const float* __restrict__ g_write, int ones, float q_scale,
+                   int share) {
     extern __shared__ float sh[];
     const int cols = kScanThreads / split;                  // value columns of this block
     const int Dp = (PER + 4) * split;                       // a staged token's channels, with the padding
@@ -128,6 +131,7 @@ linear_scan_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
         for (int i = 0; i < (MODE == 1 ? PER : 1); ++i) P[i] = 1.f;
     }
     const float fixed = gate == 0 ? decay[h] : 0.f;
+    const int hD = h / share * D;                           // this head's channels of q and of k
 
     // groups of eight consecutive channels (or value columns) of one staged token
     const int dg = (D + 7) / 8, vg = (cols + 7) / 8;
@@ -140,7 +144,7 @@ linear_scan_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
             const int g = threadIdx.x + u * kScanThreads;
             if (g < n * dg) {
                 const int j = g / dg, d = (g % dg) * 8;
-                const T* row = proj + (size_t)(base + j) * ld + h * D + d;
+                const T* row = proj + (size_t)(base + j) * ld + hD + d;
                 const bool whole = vec && d + 8 <= D;
                 if (whole || d + 8 <= D) {
                     if (MODE != 1) load8(raw.q[u], row + q_off, whole);      // (a segment's first walk makes no outputs)
@@ -219,8 +223,8 @@ linear_scan_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
             const int j = i / D, d = i % D;
             const T* row = proj + (size_t)(base + j) * ld;
             const int at = j * Dp + chan_slot(d, PER, split);
-            if (MODE != 1) q_sh[at] = scan_act<T>(lsb_to_float(row[q_off + h * D + d]), q_act) * q_scale;
-            const float z = lsb_to_float(row[k_off + h * D + d]);
+            if (MODE != 1) q_sh[at] = scan_act<T>(lsb_to_float(row[q_off + hD + d]), q_act) * q_scale;
+            const float z = lsb_to_float(row[k_off + hD + d]);
             if (gate == 0) {
                 a_sh[at] = fixed;
                 b_sh[at] = scan_act<T>(z, k_act);
@@ -366,7 +370,7 @@ static inline void scan_shape(int D, int* split, int* per) {
 LSB_API int lsb_linear_scan_supported(int D) { return D > 0 && D <= 32 * 32; }
 
 // g_keep, g_write [tokens, heads]: gate 2 only.  ones: see above.  The state is [slots, heads, V + ones, D],
-// out [tokens, heads, V + ones].
+// out [tokens, heads, V + ones].  key_heads: heads of q and k, a divisor of heads.
 // seg_len > 0 with scratch given: portions longer than a segment are walked in segments side by
 // side (see above); seg_state [requests * max_segs, heads, V, D] and seg_decay [requests * max_segs,
 // heads, D] with max_segs = ceil(max_q_len / seg_len).
@@ -375,9 +379,10 @@ LSB_API int lsb_linear_scan(const void* proj, int dtype, long long ld, int q_off
                             const float* floor_, int q_act, int k_act, int v_act, float* state,
                             int n_slots, const int* q_start, const int* table_rows, int n_requests,
                             float* out, int seg_len, int max_q_len, float* seg_state, float* seg_decay,
-                            const float* g_keep, const float* g_write, int ones, float q_scale,
+                            const float* g_keep, const float* g_write, int ones, float q_scale, int key_heads,
                             cudaStream_t stream) {
     if (n_requests <= 0) return 0;
+    if (key_heads <= 0 || heads % key_heads || (gate == 1 && key_heads != heads)) return (int)cudaErrorInvalidValue;
     if (heads <= 0 || V <= 0 || !lsb_linear_scan_supported(D) || heads > 65535 || n_requests > 65535)
         return (int)cudaErrorInvalidValue;
     if ((gate == 0 && !decay) || (gate == 1 && !floor_) || (gate == 2 && (!g_keep || !g_write)) || gate < 0 || gate > 2)
@@ -406,7 +411,7 @@ LSB_API int lsb_linear_scan(const void* proj, int dtype, long long ld, int q_off
         int rc = lsb_launch(linear_scan_kernel<T, PER, MODE>, grid, dim3(kScanThreads), smem, stream, 1, \
                           (const T*)proj, ld, q_off, k_off, v_off, heads, D, V, gate, decay, f_bias,  \
                           floor_, q_act, k_act, v_act, state, n_slots, q_start, table_rows, out, split, vec, \
-                          seg_len, max_segs, seg_state, seg_decay, g_keep, g_write, ones, q_scale);   \
+                          seg_len, max_segs, seg_state, seg_decay, g_keep, g_write, ones, q_scale, heads / key_heads); \
         if (rc) return rc;                                                                            \
     } while (0)
 #define LSB_SCAN_PER(MODE)                                                                            \
@@ -431,4 +436,37 @@ LSB_API int lsb_linear_scan(const void* proj, int dtype, long long ld, int q_off
 #undef LSB_SCAN_PER
 #undef LSB_SCAN_LAUNCH
     return 0;
+}
+
+// Queries and keys of a fixed-decay memory turned by their positions, in place in the 32-bit rows of the
+// projection: pairs (i, i + dims / 2) of the first `dims` channels of every head by pos * inv_freq[i], angle
+// and rotation in 32-bit.
+constexpr int kTurnMaxHalf = 512;
+
+__global__ void __launch_bounds__(256) turn_heads_kernel(float* __restrict__ proj, long long ld, int q_off, int k_off, int heads,
+                                                         int D, int dims, const float* __restrict__ inv_freq,
+                                                         const int* __restrict__ positions) {
+    __shared__ float cs[kTurnMaxHalf], sn[kTurnMaxHalf];
+    lsb_pdl_launch_dependents();
+    const int t = blockIdx.x, half = dims >> 1;
+    const float pos = (float)positions[t];                  // (metadata: on the device before the step's first kernel)
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &sn[i], &cs[i]);
+    __syncthreads();
+    lsb_pdl_wait();
+    float* row = proj + (size_t)t * ld;
+    for (int w = threadIdx.x; w < 2 * heads * half; w += blockDim.x) {
+        const int hh = w / half, i = w - hh * half;
+        float* at = row + (hh < heads ? q_off + hh * D : k_off + (hh - heads) * D) + i;
+        const float a = at[0], b = at[half];
+        at[0] = a * cs[i] - b * sn[i];
+        at[half] = b * cs[i] + a * sn[i];
+    }
+}
+
+LSB_API int lsb_turn_heads(float* proj, long long ld, int q_off, int k_off, int heads, int D, int dims, const float* inv_freq,
+                           const int* positions, int tokens, cudaStream_t stream) {
+    if (tokens <= 0 || dims == 0) return 0;
+    if (heads <= 0 || D <= 0 || dims < 0 || dims % 2 || dims > D || dims / 2 > kTurnMaxHalf) return (int)cudaErrorInvalidValue;
+    return lsb_launch(turn_heads_kernel, dim3(tokens), dim3(256), 0, stream, 1, proj, ld, q_off, k_off, heads, D, dims, inv_freq,
+                      positions);
 }

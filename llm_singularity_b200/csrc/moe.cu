@@ -3,6 +3,7 @@
 //   moe_route    per token: scores from the 32-bit router logits (sigmoid, softmax over all experts,
 //                or softmax over the chosen alone), the `top` largest (the lower index wins a tie),
 //                optionally divided by their sum -> ids [T, top], weights [T, top].
+//                (or no router: the experts of a token stand in a table's row of its id, all with one weight)
 //   moe_align    the (token, choice) pairs sorted by expert into rows; each expert's rows start
 //                on a multiple of the row tile, so a tile of rows belongs to one expert.  Writes
 //                pos [T * top] (the row of each pair), row_token / row_scale [capacity] (-1 / 0 in
@@ -57,6 +58,14 @@ struct RouteOpts {
 };
 
 constexpr int kMaxTop = 32;
+
+// Experts chosen by the token's id: table [rows, top], every choice with the same weight.
+struct TokenRows {
+    const int* table;
+    const int* token_ids;
+    int rows;
+    float weight;
+};
 
 // One warp chooses for one token, up to 128 experts: the logits in registers, four a lane, a chosen one struck
 // out; lane k keeps what the k-th choice was.
@@ -181,7 +190,7 @@ __global__ void __launch_bounds__(1024, 1)
 moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top, int E,
                  int cap_tiles, int tile, int* __restrict__ pos, int* __restrict__ row_token,
                  float* __restrict__ row_scale, int* __restrict__ tile_expert,
-                 const float* __restrict__ logits, RouteOpts ro) {
+                 const float* __restrict__ logits, RouteOpts ro, TokenRows by) {
     extern __shared__ int shi[];
     int* counts = shi;                  // E
     int* starts = shi + E;              // E + 1, in rows
@@ -191,6 +200,16 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
         for (int t = threadIdx.x >> 5; t < n / top; t += blockDim.x >> 5)
             route_token(logits + (size_t)t * ro.ld, E, top, ro, ids + (size_t)t * top, wts + (size_t)t * top,
                         threadIdx.x & 31);
+        __syncthreads();
+    }
+    if (by.table) {                     // no router: a token's experts are its id's row of the table
+        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+            const int tok = by.token_ids[i / top];
+            const bool known = tok >= 0 && tok < by.rows;
+            if (!known) lsb_set_status(LSB_BAD_TOKEN);
+            ids[i] = known ? by.table[(size_t)tok * top + i % top] : -1;
+            wts[i] = by.weight;
+        }
         __syncthreads();
     }
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
@@ -415,18 +434,21 @@ LSB_API int lsb_moe_route(const float* logits, int ld, int n_tokens, int E, int 
                       dim3(32 * warps_per_block), 0, stream, 1, logits, n_tokens, E, top, ro, ids, wts);
 }
 
-// logits given (32-bit [tokens, E]): ids and wts are chosen here first (see lsb_moe_route) and written
+// logits given (32-bit [tokens, E]): ids and wts are chosen here first (see lsb_moe_route) and written;
+// table given ([table_rows, top]): they are read from the row of each token's id, the weights all table_weight
 LSB_API int lsb_moe_align(int* ids, float* wts, int n_tokens, int top, int E, int cap_tiles,
                           int tile, int* pos, int* row_token, float* row_scale, int* tile_expert,
                           const float* logits, int ld, int score, int renorm, const float* bias, int joins, float scale, float eps,
-                          cudaStream_t stream) {
+                          const int* table, const int* token_ids, int table_rows, float table_weight, cudaStream_t stream) {
     const RouteOpts ro = {score, renorm, bias, scale, eps, joins, ld};
+    const TokenRows by = {table, token_ids, table_rows, table_weight};
+    if (table && (logits || !token_ids || table_rows <= 0)) return (int)cudaErrorInvalidValue;
     if (n_tokens <= 0) return 0;
     const long long n = (long long)n_tokens * top;
     if (E <= 0 || E > 8192 || tile <= 0 || cap_tiles < (n + tile - 1) / tile + E) return (int)cudaErrorInvalidValue;
     if (logits && (top > kMaxTop || top > E || score < 0 || score > 2 || ld < E)) return (int)cudaErrorInvalidValue;
     return lsb_launch(moe_align_kernel, dim3(1), dim3(1024), (size_t)(2 * E + 1) * sizeof(int), stream, 1,
-                      ids, wts, (int)n, top, E, cap_tiles, tile, pos, row_token, row_scale, tile_expert, logits, ro);
+                      ids, wts, (int)n, top, E, cap_tiles, tile, pos, row_token, row_scale, tile_expert, logits, ro, by);
 }
 
 // rows[pos[t, k]] = T(wts[t, k] * x[t]): the operand of the grouped tensor-core product, which wants

@@ -1009,7 +1009,7 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
                 value_dim: int, gate: str, decay: Optional[torch.Tensor], f_bias: Optional[torch.Tensor],
                 floor: Optional[torch.Tensor], q_act: str, k_act: str, v_act: str, state: torch.Tensor,
                 ctx, out: torch.Tensor, keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
-                ones: bool = False, q_scale: float = 1.0) -> None:
+                ones: bool = False, q_scale: float = 1.0, key_heads: Optional[int] = None) -> None:
     """S <- diag(a) S + b v^T, o = S^T q per head and token, each request from its slot's state
     (``state`` [slots, heads, value_dim, key_dim] 32-bit, updated in place); ``proj`` [T, columns] holds
     the projections of q at ``q_off``, of k (or the forget gate) at ``k_off`` and of v at ``v_off``;
@@ -1018,7 +1018,8 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     Gate "given": ``keep`` and ``write`` (32-bit [T, heads]) are a and the factor of b for every channel
     of a head.  ``ones``: a value column of ones rides along behind each head's ``value_dim`` columns
     (state and out then have ``value_dim + 1`` columns a head, the last one of out being the
-    running sum of b dotted with q).  ``q_scale`` multiplies q."""
+    running sum of b dotted with q).  ``q_scale`` multiplies q.  ``key_heads``: heads of q and k, shared by
+    groups of ``heads / key_heads`` heads (not with the forget gate)."""
     _req(proj, "proj", dim=2)
     _req(state, "state", torch.float32, 4)
     _req(out, "out", torch.float32, 2)
@@ -1026,7 +1027,10 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     cols = value_dim + (1 if ones else 0)
     if state.shape[1:] != (heads, cols, key_dim) or out.shape != (T, heads * cols) or ctx.n_tokens != T:
         raise KernelError("linear_scan: state, out or the step do not fit the sizes")
-    if max(q_off, k_off) + heads * key_dim > ld or v_off + heads * value_dim > ld or min(q_off, k_off, v_off) < 0:
+    key_heads = heads if key_heads is None else key_heads
+    if key_heads <= 0 or heads % key_heads or (gate == "forget" and key_heads != heads):
+        raise KernelError(f"linear_scan: {heads} heads cannot share {key_heads} heads of q and k")
+    if max(q_off, k_off) + key_heads * key_dim > ld or v_off + heads * value_dim > ld or min(q_off, k_off, v_off) < 0:
         raise KernelError("linear_scan: a projection lies outside the rows of proj")
     if gate == "given" and (keep is None or write is None):
         raise KernelError("linear_scan: given gates need keep and write")
@@ -1054,7 +1058,87 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
           _i(heads), _i(key_dim), _i(value_dim), _i(SCAN_GATES[gate]), _p(decay), _p(f_bias), _p(floor),
           _i(_SCAN_ACTS[q_act]), _i(_SCAN_ACTS[k_act]), _i(_SCAN_ACTS[v_act]), _p(state), _i(state.shape[0]),
           _p(ctx.q_start), _p(ctx.table_rows), _i(ctx.n_requests), _p(out), _i(seg), _i(ctx.max_q_len),
-          _p(seg_state), _p(seg_decay), _p(keep), _p(write), _i(1 if ones else 0), _f(q_scale), _stream(out))
+          _p(seg_state), _p(seg_decay), _p(keep), _p(write), _i(1 if ones else 0), _f(q_scale), _i(key_heads),
+          _stream(out))
+
+
+def turn_heads(proj: torch.Tensor, q_off: int, k_off: int, heads: int, key_dim: int, inv_freq: torch.Tensor, ctx) -> None:
+    """The first ``2 * len(inv_freq)`` channels of every head of q and k (``heads`` heads of ``key_dim`` from
+    ``q_off`` and ``k_off`` on in the 32-bit rows of ``proj``) turned by the token's position, in place: pairs
+    (i, i + half) by ``pos * inv_freq[i]``."""
+    _req(proj, "proj", torch.float32, 2)
+    _req(inv_freq, "inv_freq", torch.float32, 1)
+    T, ld = proj.shape
+    dims = 2 * inv_freq.shape[0]
+    if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off) < 0 or max(q_off, k_off) + heads * key_dim > ld:
+        raise KernelError("turn_heads: proj, the heads and the step disagree")
+    _call("linear_scan", "lsb_turn_heads", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(heads), _i(key_dim), _i(dims),
+          _p(inv_freq), _p(ctx.positions), _i(T), _stream(proj))
+
+
+# ----------------------------------------------------------------- state-space memory
+def state_space_prep(proj: torch.Tensor, x_off: int, dt_off: int, channels: int, conv: torch.Tensor, conv_bias: torch.Tensor,
+                     dt_bias: torch.Tensor, a_log: torch.Tensor, conv_state: Optional[torch.Tensor], ctx, u: torch.Tensor,
+                     fades: torch.Tensor) -> None:
+    """From the 32-bit rows of ``proj``: u [T, channels] = silu(conv_bias + causal convolution of the ``channels``
+    columns from ``x_off`` on), taps ``conv`` [channels, n] whose last column meets the current token, the inputs
+    before a portion from ``conv_state`` [slots, n - 1, channels]; and per head dt = softplus(proj[:, dt_off:] +
+    dt_bias): ``fades`` [3, T, heads] receives exp(-exp(a_log) dt), dt and -exp(a_log) dt.  In a step of single
+    tokens ``conv_state`` is updated here, in others by ``state_space_output``."""
+    _req(proj, "proj", torch.float32, 2)
+    _req(u, "u", dim=2)
+    _req(fades, "fades", torch.float32, 3)
+    _req(conv, "conv", torch.float32, 2)
+    T, ld = proj.shape
+    heads, n = fades.shape[2], conv.shape[1]
+    for name, t, k in (("conv_bias", conv_bias, channels), ("dt_bias", dt_bias, heads), ("a_log", a_log, heads)):
+        _req(t, name, torch.float32, 1)
+        if t.shape[0] != k:
+            raise KernelError(f"state_space_prep: {name} must have {k} entries")
+    if (ctx.n_tokens != T or u.shape != (T, channels) or fades.shape != (3, T, heads) or conv.shape[0] != channels
+            or min(x_off, dt_off) < 0 or x_off + channels > ld or dt_off + heads > ld):
+        raise KernelError("state_space_prep: proj, u, the fades and the step do not fit the sizes")
+    slots = 1 << 30
+    if n > 1:
+        _req(conv_state, "conv_state", torch.float32, 3)
+        if conv_state.shape[1:] != (n - 1, channels):
+            raise KernelError(f"state_space_prep: conv_state must be [slots, {n - 1}, {channels}]")
+        slots = conv_state.shape[0]
+    _call("state_space", "lsb_state_space_prep", _p(proj), _ll(ld), _i(x_off), _i(dt_off), _i(T), _i(channels), _i(heads), _i(n),
+          _p(conv), _p(conv_bias), _p(dt_bias), _p(a_log), _p(conv_state if n > 1 else None), _i(slots), _p(ctx.token_req),
+          _p(ctx.q_start), _p(ctx.table_rows), _p(u), _i(_dt(u)), _p(fades[0]), _p(fades[1]), _p(fades[2]),
+          _i(1 if ctx.max_q_len == 1 and n > 1 else 0), _stream(u))
+
+
+def state_space_output(y: torch.Tensor, proj: torch.Tensor, x_off: int, u: torch.Tensor, d: torch.Tensor, weight: torch.Tensor,
+                       heads: int, groups: int, eps: float, taps: int, conv_state: Optional[torch.Tensor], ctx,
+                       out: torch.Tensor) -> None:
+    """v = (y + d[head] * u) * silu(proj's first columns) over the ``heads * V`` columns of ``y`` (32-bit, the walk's
+    read-out; ``u``'s first columns are the convolved x); out = v divided by the root mean square of its part
+    (``groups`` equal parts of the row) times ``weight``.  In steps that bring portions the convolution's inputs in
+    ``conv_state`` are replaced by the portions' last ``taps - 1``."""
+    _req(y, "y", torch.float32, 2)
+    _req(proj, "proj", torch.float32, 2)
+    _req(out, "out", dim=2)
+    _req(u, "u", out.dtype, 2)
+    T, inner = y.shape
+    for name, t, k in (("d", d, heads), ("weight", weight, inner)):
+        _req(t, name, torch.float32, 1)
+        if t.shape[0] != k:
+            raise KernelError(f"state_space_output: {name} must have {k} entries")
+    channels = u.shape[1]
+    if (ctx.n_tokens != T or out.shape != y.shape or proj.shape[0] != T or u.shape[0] != T or channels < inner or inner % heads
+            or groups <= 0 or inner % groups or inner > proj.shape[1] or x_off + channels > proj.shape[1]):
+        raise KernelError("state_space_output: y, proj, u, out and the step do not fit the sizes")
+    update = taps > 1 and ctx.max_q_len > 1
+    if update:
+        _req(conv_state, "conv_state", torch.float32, 3)
+        if conv_state.shape[1:] != (taps - 1, channels):
+            raise KernelError(f"state_space_output: conv_state must be [slots, {taps - 1}, {channels}]")
+    _call("state_space", "lsb_state_space_output", _p(y), _p(proj), _ll(proj.shape[1]), _i(x_off), _p(u), _i(channels), _p(d),
+          _p(weight), _i(T), _i(heads), _i(inner // heads), _i(groups), _f(eps), _i(taps if update else 0),
+          _p(conv_state if update else None), _i(conv_state.shape[0] if update else 0), _p(ctx.token_req), _p(ctx.q_start),
+          _p(ctx.table_rows), _p(out), _i(_dt(out)), _stream(out))
 
 
 # --------------------------------------------------------------------- latent attention
@@ -1308,6 +1392,43 @@ def stream_norm(residual: torch.Tensor, y: Optional[torch.Tensor], post_weight: 
           _i(T), _i(H), _stream(residual))
 
 
+def join_norm(residual: torch.Tensor, ys, scales, bias: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
+              copy: Optional[torch.Tensor], pos: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None) -> None:
+    """residual += unit(v) * weight in place (32-bit), copy <- residual in its type (None: no copy), with
+    v = sum_b scales[b] * ys[b] + bias; or, with ``pos`` and ``wts`` [T, top], v[t] = sum_k wts[t, k] *
+    ys[0][pos[t * top + k]] (+ bias).  unit(z) = z / sqrt(mean(z^2) + eps); everything in 32-bit."""
+    _req(residual, "residual", torch.float32, 2)
+    _req(weight, "weight", torch.float32, 1)
+    T, H = residual.shape
+    n = len(ys)
+    if n == 0 or n != len(scales) or n > _lib("output_norm").lsb_join_max_terms() or weight.shape[0] != H:
+        raise KernelError(f"join_norm: {n} terms with {len(scales)} factors, weight {tuple(weight.shape)}")
+    top = capacity = 0
+    if pos is not None:
+        _req(pos, "pos", torch.int32, 1)
+        _req(wts, "wts", torch.float32, 2)
+        top, capacity = wts.shape[1], ys[0].shape[0]
+        if n != 1 or wts.shape[0] != T or pos.shape[0] != T * top:
+            raise KernelError("join_norm: expert rows need a place and a weight for every choice of every token")
+    for y in ys:
+        _req(y, "term", ys[0].dtype, 2)
+        if y.shape[1] != H or (pos is None and y.shape[0] != T):
+            raise KernelError("join_norm: a term does not fit the stream")
+    if bias is not None:
+        _req(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != H:
+            raise KernelError("join_norm: the bias must have one number a column")
+    if copy is not None:
+        _req(copy, "copy", dim=2)
+        if copy.shape != (T, H):
+            raise KernelError("join_norm: copy has another shape than the stream")
+    yp = (ctypes.c_void_p * n)(*[_p(y).value for y in ys])
+    sc = (ctypes.c_float * n)(*[float(x) for x in scales])
+    _call("output_norm", "lsb_join_norm", _p(residual), yp, sc, _i(n), _i(_dt(ys[0])), _p(bias), _p(pos), _p(wts), _i(top),
+          _i(capacity), _p(weight), _f(eps), _p(copy), _i(_dt(copy) if copy is not None else _F32), _i(T), _i(H),
+          _stream(residual))
+
+
 def stream_centred_norm(residual: torch.Tensor, y: Optional[torch.Tensor], post_weight: Optional[torch.Tensor],
                         post_bias: Optional[torch.Tensor], post_eps: float, mult: float, rows: Optional[torch.Tensor],
                         next_weight: Optional[torch.Tensor], next_bias: Optional[torch.Tensor], next_eps: float,
@@ -1377,7 +1498,7 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
                    inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, pairing: str = "half",
                    store: bool = True, norm_all: bool = False, v_unit: bool = False,
                    v_first: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
-                   maps: int = 1) -> None:
+                   maps: int = 1, qk_unit: bool = False) -> None:
     """From the rows of ``proj`` (q at ``q_off``, k at ``k_off``, v at ``v_off``) to queries in ``q_out``
     [T, nh * dk] and keys and values in this step's cache places: biases, a norm per head of q and k
     (one weight of head size each), the query temperature ``1 + coef * ln(floor((pos + 1) / every) + 1)``
@@ -1387,7 +1508,8 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
     ``v_first`` [T, nkv * dv] (rows may be strided) with ``v_lambda`` (one 32-bit number on the device): the
     values are mixed with those another layer made of the same tokens, v <- (1 - lambda) v + lambda v_first,
     and cached so.  ``maps``: every query and key head is that many parts of ``dk`` side by side, each normed
-    and rotated as a head of its own; q_out is then [T, nh * maps * dk] and a cached key maps * dk long."""
+    and rotated as a head of its own; q_out is then [T, nh * maps * dk] and a cached key maps * dk long.
+    ``qk_unit``: every head of q and k is divided by its root mean square (eps ``norm_eps``, no weight)."""
     _req(proj, "proj", dim=2)
     _req(q_out, "q_out", proj.dtype, 2)
     T, ld = proj.shape
@@ -1412,6 +1534,8 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
         if rotary_dim % 2 or rotary_dim > dk or inv_freq.shape[0] != rotary_dim // 2:
             raise KernelError("attention_prep: rotary_dim must be even, at most the key size, with rotary_dim / 2 "
                               "frequencies")
+    if qk_unit and (q_norm is not None or k_norm is not None):
+        raise KernelError("attention_prep: a norm without a weight beside one with")
     if norm_all and (q_norm is None) != (k_norm is None):
         raise KernelError("attention_prep: a norm over all heads needs both weights")
     v_first_ld = 0
@@ -1424,7 +1548,8 @@ def attention_prep(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: i
     _check_kv_cache(cache, nkv, maps * dk, dv, proj.dtype)
     _call("attention_prep", "lsb_attention_prep", _p(proj), _i(_dt(proj)), _ll(ld), _i(q_off), _i(k_off), _i(v_off),
           _i(T), _i(nh), _i(nkv), _i(dk), _i(dv), _p(q_bias), _p(k_bias), _p(v_bias), _p(q_norm), _p(k_norm),
-          _f(norm_eps), _i(1 if norm_all else 0), _i(1 if v_unit else 0), _i(maps), _f(temp_coef), _i(temp_every), _p(inv_freq if rotary_dim else None), _i(rotary_dim),
+          _f(norm_eps), _i(1 if norm_all else 0), _i(1 if v_unit else 0), _i(1 if qk_unit else 0), _i(maps), _f(temp_coef),
+          _i(temp_every), _p(inv_freq if rotary_dim else None), _i(rotary_dim),
           _i(_PAIRINGS[pairing]), _p(ctx.positions), _p(ctx.token_req), _p(ctx.table_rows), _p(cache.block_table),
           _i(cache.block_table.shape[1]), _p(q_out), _p(cache.k_pages), _p(cache.v_pages), _i(cache.page_size),
           _i(cache.k_pages.shape[0]), _i(1 if store else 0), _p(v_first), _ll(v_first_ld), _p(v_lambda), _stream(proj))
@@ -1436,13 +1561,14 @@ DV_TENSOR_CORES = True          # bfloat16 heads of multiples of 16 up to 128 on
 
 def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cache, scale: float, window: int,
                  chunk: int, gate: Optional[torch.Tensor], out: torch.Tensor, sink: bool = False,
-                 gate_per_head: bool = False, softcap: float = 0.0, linear_bias: bool = False) -> None:
+                 gate_per_head: bool = False, softcap: float = 0.0, linear_bias: bool = False,
+                 sink_logit: Optional[torch.Tensor] = None) -> None:
     """Softmax attention of this step's queries ``q`` [T, nh * dk] over their requests' cached keys (size
     dk) and values (size dv): a query at position p sees ``[lo, p]`` with lo the larger of
     ``p - window + 1`` (window > 0) and the start of p's chunk of ``chunk`` positions (chunk > 0).
     ``gate`` [T, nh * dv] (rows may be strided): out *= sigmoid(gate); with ``gate_per_head`` it is
     [T, nh], one number per head.  ``sink``: one is added to the softmax's denominator (a place with
-    score 0 and no value).  ``softcap`` > 0: a scaled score s becomes softcap * tanh(s / softcap).
+    score 0 and no value); with ``sink_logit`` (32-bit [nh]) it is exp(sink_logit[h]), not scaled.  ``softcap`` > 0: a scaled score s becomes softcap * tanh(s / softcap).
     ``linear_bias``: head h's score for the key at distance d loses 2^(-8 (h + 1) / nh) * d (after the cap).
 
     bfloat16 with both sizes multiples of 16 up to 128 runs on the tensor cores (prompt portions in
@@ -1465,6 +1591,10 @@ def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cach
         gate_stride = gate.stride(0)
     flags = (1 if sink else 0) | (2 if gate is not None and gate_per_head else 0) | (4 if linear_bias else 0)
     softcap = float(softcap or 0.0)
+    if sink_logit is not None:
+        _req(sink_logit, "sink_logit", torch.float32, 1)
+        if sink_logit.shape[0] != nh or not sink:
+            raise KernelError("attention_dv: the sink's scores are one number a head of an attention with a sink")
     if softcap < 0:
         raise KernelError("attention_dv: the cap must be positive (0: none)")
     _check_kv_cache(cache, nkv, dk, dv, q.dtype)
@@ -1473,7 +1603,7 @@ def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cach
     # where they all come before the portions (as the scheduler puts them), go on below
     n_req, max_q = ctx.n_requests, ctx.max_q_len
     if (USE_TCGEN05_ATTENTION and DV_TENSOR_CORES and q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128)
-            and not chunk and (gate is None or gate_per_head) and ctx.max_q_len >= 128
+            and not chunk and (gate is None or gate_per_head) and ctx.max_q_len >= 128 and scale > 0
             and cache.page_size in (8, 16, 32, 64)
             and _lib("attention_tc5").lsb_prefill_attention_tc5_supported(
                 _p(q), _i(q.shape[1]), _p(cache.k_pages), _p(cache.v_pages), _i(nh), _i(nkv), _i(dk), _i(cache.page_size))):
@@ -1486,7 +1616,7 @@ def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cach
                   _p(cache.block_table), _i(cache.block_table.shape[1]), _p(out), _i(ctx.n_requests - first),
                   _i(ctx.max_q_len), _i(nh), _i(nkv), _i(dk), _i(cache.page_size), _i(cache.k_pages.shape[0]), _f(scale),
                   _i(window), _i(0), _i(1 if sink else 0), _p(gate), _ll(gate_stride), _f(softcap),
-                  _i(1 if linear_bias else 0), _stream(out))
+                  _i(1 if linear_bias else 0), _p(sink_logit), _stream(out))
             if first == 0:
                 return
             n_req, max_q = first, 1
@@ -1509,13 +1639,13 @@ def attention_dv(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cach
               _p(ctx.kv_len), _p(ctx.table_rows), _p(cache.block_table), _i(cache.block_table.shape[1]), _p(gate),
               _ll(gate_stride), _p(out), _i(n_req), _i(max_q), _i(nh), _i(nkv), _i(dk), _i(dv),
               _i(cache.page_size), _i(cache.k_pages.shape[0]), _f(scale), _i(window), _i(chunk), _i(num_sms(q.device)),
-              _i(DV_BLOCK_SHAPE), _p(scratch), _i(flags), _f(softcap), _stream(out))
+              _i(DV_BLOCK_SHAPE), _p(scratch), _i(flags), _f(softcap), _p(sink_logit), _stream(out))
         return
     _call("attention_dv", "lsb_attention_dv_generic", _p(q), _p(cache.k_pages), _p(cache.v_pages), _p(ctx.q_start),
           _p(ctx.kv_len), _p(ctx.table_rows), _p(cache.block_table), _i(cache.block_table.shape[1]), _p(gate),
           _ll(gate_stride), _p(out), _i(_dt(q)), _i(n_req), _i(max_q), _i(nh), _i(nkv), _i(dk),
           _i(dv), _i(cache.page_size), _i(cache.k_pages.shape[0]), _f(scale), _i(window), _i(chunk), _i(flags), _f(softcap),
-          _stream(out))
+          _p(sink_logit), _stream(out))
 
 
 def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, cache, scale: float, window: int,
@@ -1580,9 +1710,13 @@ def attention_diff(q: torch.Tensor, nh: int, nkv: int, dk: int, dv: int, ctx, ca
               _i(DV_BLOCK_SHAPE), _p(scratch), _stream(out))
 
 
-def branch_sum(ys, scales, out: torch.Tensor) -> None:
-    """out = sum_b scales[b] * ys[b], summed in 32-bit (mixers side by side whose results are added
-    with fixed factors)."""
+def branch_sum(ys, scales, out: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
+    """out = sum_b scales[b] * ys[b] (+ ``bias``, 32-bit, one number a column), summed in 32-bit (mixers side
+    by side whose results are added with fixed factors)."""
+    if bias is not None:
+        _req(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != out.shape[1]:
+            raise KernelError("branch_sum: the bias must have one number a column")
     n = len(ys)
     if n == 0 or len(scales) != n:
         raise KernelError("branch_sum: one factor per branch")
@@ -1593,7 +1727,7 @@ def branch_sum(ys, scales, out: torch.Tensor) -> None:
             raise KernelError("branch_sum: every branch must have out's shape")
     yp = (ctypes.c_void_p * n)(*[_p(y).value for y in ys])
     sc = (ctypes.c_float * n)(*[float(x) for x in scales])
-    _call("sandwich", "lsb_branch_sum", yp, sc, _i(n), _p(out), _i(_dt(out)), _i(out.shape[0]), _i(out.shape[1]),
+    _call("sandwich", "lsb_branch_sum", yp, sc, _i(n), _p(bias), _p(out), _i(_dt(out)), _i(out.shape[0]), _i(out.shape[1]),
           _stream(out))
 
 
@@ -1748,25 +1882,28 @@ def delta_scan(form: str, vecs: torch.Tensor, scal: Optional[torch.Tensor], vals
 _DELTA_GATES = {"none": 0, "sigmoid": 1, "silu": 2}
 
 
-def delta_output(x: torch.Tensor, weight: torch.Tensor, heads: int, eps: float, gate: Optional[torch.Tensor],
+def delta_output(x: torch.Tensor, weight: Optional[torch.Tensor], heads: int, eps: float, gate: Optional[torch.Tensor],
                  gate_act: str, out: torch.Tensor) -> None:
     """out = each head of the 32-bit row ``x`` [T, heads * V] divided by its root mean square, times ``weight``
-    (its index taken modulo its length: one weight per head, or one over the row), times sigmoid or silu of
-    ``gate`` [T, heads * V] (rows may be strided)."""
+    (None: no weight; its index taken modulo its length: one weight per head, or one over the row), times
+    sigmoid or silu of ``gate`` [T, heads * V] (in out's type or 32-bit, rows may be strided)."""
     _req(x, "x", torch.float32, 2)
-    _req(weight, "weight", torch.float32, 1)
     _req(out, "out", dim=2)
     T, n = x.shape
-    if out.shape != (T, n) or heads <= 0 or n % heads or n % weight.shape[0] or gate_act not in _DELTA_GATES:
+    w_len = 1
+    if weight is not None:
+        _req(weight, "weight", torch.float32, 1)
+        w_len = weight.shape[0]
+    if out.shape != (T, n) or heads <= 0 or n % heads or n % w_len or gate_act not in _DELTA_GATES:
         raise KernelError("delta_output: shapes disagree")
     gate_stride = 0
     if gate is not None:
-        _req(gate, "gate", out.dtype, 2, contiguous=False)
+        _req(gate, "gate", None if gate.dtype == torch.float32 else out.dtype, 2, contiguous=False)
         if gate.shape != (T, n) or gate.stride(1) != 1:
             raise KernelError("delta_output: the gate must have x's shape and unit column stride")
         gate_stride = gate.stride(0)
-    _call("delta_rule", "lsb_delta_output", _p(x), _p(weight), _i(weight.shape[0]), _p(gate), _ll(gate_stride),
-          _i(_DELTA_GATES[gate_act] if gate is not None else 0), _p(out), _i(_dt(out)), _i(T), _i(heads), _i(n // heads),
+    _call("delta_rule", "lsb_delta_output", _p(x), _p(weight), _i(w_len), _p(gate), _ll(gate_stride),
+          _i(_DELTA_GATES[gate_act] if gate is not None else 0), _i(1 if gate is not None and gate.dtype == torch.float32 else 0), _p(out), _i(_dt(out)), _i(T), _i(heads), _i(n // heads),
           _f(eps), _stream(out))
 
 
@@ -1897,23 +2034,33 @@ def moe_routed_experts(x: torch.Tensor, logits: torch.Tensor, top: int, score: s
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, activation: str, weight_on: str, out: torch.Tensor, route=None,
                 limit: float = 0.0, add: Optional[torch.Tensor] = None, gated: bool = True,
-                add_gate: Optional[torch.Tensor] = None) -> None:
+                add_gate: Optional[torch.Tensor] = None, by_token=None, open_sum: bool = False):
     """out[t] = sum over k of down_e(act(gate_e u) * up_e u), e = ids[t, k], with u = weights[t, k] * x[t]
     (``weight_on`` "input") or u = x[t] and the sum weighted ("output"); plus ``add[t]`` if given (a shared
     expert's rows, or a callable that makes them: it is called behind the experts' products), in the same
     32-bit sum, times sigmoid(``add_gate[t, 0]``) if that is given (32-bit, rows may be strided).
     ``w_gate_up`` [E, 2F, H] has rows alternating gate_i, up_i; ``w_down`` [E, H, F].  ``gated`` False: the
-    experts are down_e(act(up_e u)) and ``w_gate_up`` is [E, F, H], the up matrices alone."""
+    experts are down_e(act(up_e u)) and ``w_gate_up`` is [E, F, H], the up matrices alone.
+
+    ``by_token = (table, token_ids)``: the experts are those that row ``token_ids[t]`` of the int32 ``table`` [R, top]
+    names, all with the weight 1 / top; ids and weights are filled in.  ``open_sum``: nothing is summed and ``out``
+    may be None; what comes back is (y, pos): the experts' rows and where each (token, choice) has its own."""
     _req(x, "x", dim=2)
     _req(ids, "ids", torch.int32, 2)
     _req(weights, "weights", torch.float32, 2)
     _req(w_gate_up, "w_gate_up", x.dtype, 3)
     _req(w_down, "w_down", x.dtype, 3)
-    _req(out, "out", x.dtype, 2)
     T, H = x.shape
+    if open_sum:
+        if weight_on != "output" or add is not None:
+            raise KernelError("moe_experts: rows that are summed elsewhere carry their weights on the output")
+    else:
+        _req(out, "out", x.dtype, 2)
+        if out.shape != (T, H):
+            raise KernelError("moe_experts: shapes disagree")
     E, N_up, _ = w_gate_up.shape
     F, top = N_up // 2 if gated else N_up, ids.shape[1]
-    if w_gate_up.shape != (E, 2 * F if gated else F, H) or w_down.shape != (E, H, F) or out.shape != (T, H) \
+    if w_gate_up.shape != (E, 2 * F if gated else F, H) or w_down.shape != (E, H, F) \
             or ids.shape[0] != T or weights.shape != ids.shape or weight_on not in ("input", "output"):
         raise KernelError("moe_experts: shapes disagree")
     if gated:
@@ -1933,13 +2080,20 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         tile = MOE_ROW_TILE or (16 if mean <= 8 else 32 if mean <= 16 else 64 if mean <= 32 else 128)
     cap_tiles = -(-T * top // tile) + E
     dev = x.device
+    table = token_ids = None
+    if by_token is not None:
+        table, token_ids = by_token
+        _req(table, "table", torch.int32, 2)
+        _req(token_ids, "token_ids", torch.int32, 1)
+        if table.shape[1] != top or token_ids.shape[0] != T or route is not None:
+            raise KernelError("moe_experts: the table must have `top` columns, and the step a token id per row")
     pos = torch.empty(T * top, dtype=torch.int32, device=dev)
     row_token = torch.empty(cap_tiles * tile, dtype=torch.int32, device=dev)
     row_scale = torch.empty(cap_tiles * tile, dtype=torch.float32, device=dev)
     tile_expert = torch.empty(cap_tiles, dtype=torch.int32, device=dev)
     hidden = torch.empty(cap_tiles * tile, F, dtype=x.dtype, device=dev)
     y = torch.empty(cap_tiles * tile, H, dtype=x.dtype if tc else torch.float32, device=dev)
-    s = _stream(out)
+    s = _stream(x)
     on_input = 1 if weight_on == "input" else 0
     # a shared expert's rows: on a stream of their own in a step of few tokens, else made behind the experts'
     # products (its own products' weights are then the last streamed before the next layer's, which they ask
@@ -1951,7 +2105,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         raise KernelError("moe_experts: the router's logits must be [tokens, experts]")
     _call("moe", "lsb_moe_align", _p(ids), _p(weights), _i(T), _i(top), _i(E), _i(cap_tiles), _i(tile), _p(pos),
           _p(row_token), _p(row_scale), _p(tile_expert), _p(r_logits), _i(E if r_logits is None else r_logits.shape[1]),
-          _i(r_score), _i(r_renorm), *_route_options(E, r_bias, r_scale, r_eps, r_joins), s)
+          _i(r_score), _i(r_renorm), *_route_options(E, r_bias, r_scale, r_eps, r_joins), _p(table), _p(token_ids),
+          _i(table.shape[0] if table is not None else 0), _f(1.0 / top), s)
     if tc:
         rows = torch.empty(cap_tiles * tile, H, dtype=x.dtype, device=dev)
         _call("moe", "lsb_moe_gather", _p(x), _i(_dt(x)), _p(pos), _p(weights), _i(on_input), _i(T), _i(top),
@@ -1966,6 +2121,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
               _p(tile_expert), _i(cap_tiles), _p(hidden), _i(F), _i(H), _i(act), _f(limit), _i(0 if gated else 1), s)
         _call("moe", "lsb_moe_down", _p(hidden), _i(_dt(x)), _p(row_token), _p(w_down), _p(tile_expert), _i(cap_tiles),
               _p(y), _i(H), _i(F), s)
+    if open_sum:
+        return y, pos
     if add_join is not None:
         add = add_join()
     if add is not None:

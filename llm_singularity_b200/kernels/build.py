@@ -46,6 +46,8 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     "latent_tc": "latent_tc.cu",
     "moe": "moe.cu",
     "sandwich": "sandwich.cu",
+    "output_norm": "output_norm.cu",
+    "state_space": "state_space.cu",
     "attention_prep": "attention_prep.cu",
     "attention_dv": "attention_dv.cu",
     "attention_diff": "attention_diff.cu",

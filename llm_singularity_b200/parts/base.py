@@ -41,7 +41,8 @@ class ParamSpec:
     role: ``matrix`` and ``table`` are matrix-product operands and live in the
     compute dtype; ``vector`` (norm weights and the like) is kept in 32-bit;
     ``int_table`` is kept as int32.
-    init: ``normal`` -> N(0, std); ``ones`` -> 1 + N(0, noise).
+    init: ``normal`` -> N(0, std); ``ones`` -> 1 + N(0, noise); of an integer table ``distinct:<n>`` -> rows of
+    different numbers below n (``normal``: zeros).
     """
 
     shape: Tuple[int, ...]
@@ -281,6 +282,9 @@ class Part:
     # (any other gets the finished rows).  A norm with ``foldable`` has ``fold() -> (weight, eps)``.
     # A block with ``folds_next`` takes ``next_norm`` in ``forward`` (the norm its output will meet
     # first) and tells through ``first_norm()`` which norm of its own the block before may fold.
+    # ``opens_sum``: ``forward`` takes ``open_sum=True`` and may then hand back its result as a sum still to be
+    # formed (``parts.norm``: ``BranchSum``, ``ExpertRows``), for a caller whose next kernel forms it on the way.
+    opens_sum = False
     folds_norm = False
     takes_unnormed = False
     foldable = False

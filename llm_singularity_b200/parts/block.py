@@ -261,3 +261,49 @@ class SandwichBlock(Part):
             return self.mixer_post_norm.pending(y, mult)
         h = self.ffn_norm.add_norm(residual, self.mixer_post_norm.pending(y, mult))
         return self.ffn_post_norm.pending(self.ffn.forward(h, ctx), mult)
+
+
+@register_block("output_norm")
+class OutputNormBlock(Part):
+    """``x += norm1(mixer(x)); x += norm2(ffn(x))``: the sublayers read the stream itself and a norm stands
+    behind each.  The stream is 32-bit and updated in place; the norm behind a sublayer, the sum and the
+    rounded copy that the next products read are one kernel, which also forms what a sublayer leaves open (the
+    weighted sum of mixers side by side, the sum over a token's experts).  ``ffn`` None: no second step.
+
+    What it hands on is a ``StreamCopy``: nothing pending, and the copy for whoever reads next."""
+
+    graph_safe = True
+    kernels = ("output_norm", "rownorm")
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.mixer = MIXERS.build(spec.mixer, rt)
+        self.mixer_norm = NORMS.build(spec.mixer_norm, rt)
+        self.ffn = FEED_FORWARDS.build(spec.ffn, rt) if spec.ffn is not None else None
+        self.ffn_norm = NORMS.build(spec.ffn_norm, rt) if spec.ffn is not None else None
+        for n in (self.mixer_norm, self.ffn_norm):
+            if n is not None and not hasattr(n, "join"):
+                raise ValueError(f"a norm of kind '{n.spec.kind}' cannot stand behind a sublayer and join the stream (no join)")
+
+    def children(self) -> Dict[str, Part]:
+        c = {"mixer": self.mixer, "mixer_norm": self.mixer_norm}
+        if self.ffn is not None:
+            c.update(ffn=self.ffn, ffn_norm=self.ffn_norm)
+        return c
+
+    def forward(self, residual: torch.Tensor, pending, ctx, cache, writes_cache: bool = True):
+        if isinstance(pending, StreamCopy):
+            h = pending.values
+        elif pending is not None:
+            raise ValueError("a block whose sublayers read the stream itself cannot take a pending delta")
+        elif self.rt.dtype == torch.float32:
+            h = residual
+        else:
+            h = self.rt.empty(*residual.shape)
+            self.rt.ops.cast_rows(residual, h)
+        open_sum = {"open_sum": True} if self.mixer.opens_sum else {}
+        h = self.mixer_norm.join(residual, self.mixer.forward(h, ctx, cache, writes_cache, **open_sum))
+        if self.ffn is not None:
+            open_sum = {"open_sum": True} if self.ffn.opens_sum else {}
+            h = self.ffn_norm.join(residual, self.ffn.forward(h, ctx, **open_sum))
+        return StreamCopy(h)

@@ -17,7 +17,9 @@ and a gate of one number per head (``gate_per_head``); scores capped by ``cap * 
 (``ctx.lent``), a "mixed" layer caches ``(1 - lambda) v + lambda v_source``.  With ``diff`` a head attends twice
 to its values (two queries and keys side by side, one cached row) and the kernels of
 ``csrc/attention_diff.cu`` leave the normed difference of the two; the number that multiplies the second
-map is formed once at load, in 64-bit, from the layer's four vectors.
+map is formed once at load, in 64-bit, from the layer's four vectors.  Heads of q and k brought to unit rms
+without a weight (``qk_unit``), a sink whose score is a learnt number per head (``sink_logit``), and a bias of the
+output projection (``out_bias``), which a caller that forms the mixer's sum itself takes along (``open_sum``).
 
 Where the spec is what the framework's grouped attention already covers after the preparation (keys
 and values of one size, no chunks, no gate), the same attention kernels run (tensor cores for
@@ -30,6 +32,7 @@ from typing import Dict
 import torch
 
 from .base import POSITIONS, PagedKVSpec, ParamSpec, Part, register_mixer
+from .norm import BranchSum
 
 
 @register_mixer("kv_attention")
@@ -60,9 +63,16 @@ class KVAttention(Part):
             raise ValueError(f"value_mix '{self.value_mix}' is not known (source, mixed)")
         if self.value_mix and (s.qkv_bias or self.v_unit):
             raise ValueError("values that layers share are neither biased nor normed")
+        self.qk_unit = bool(getattr(s, "qk_unit", False))
+        if self.qk_unit and s.qk_norm:
+            raise ValueError("a norm of q and k without a weight beside one with")
+        self.sink_logit = bool(getattr(s, "sink_logit", False))
+        if self.sink_logit and not self.sink:
+            raise ValueError("a learnt score of a sink without a sink")
+        self.opens_sum = self.out_bias = bool(getattr(s, "out_bias", False))
         self.diff = getattr(s, "diff", None)
         if self.diff is not None and (s.qkv_bias or s.qk_norm or s.temp_every or s.out_gate or self.v_unit or self.sink
-                                      or self.softcap or self.linear_bias or self.value_mix):
+                                      or self.softcap or self.linear_bias or self.value_mix or self.qk_unit or self.out_bias):
             raise ValueError("differential attention goes with a position encoding, a window and chunks only")
         self.maps = 1 if self.diff is None else 2
         self.position = POSITIONS.build(s.position, rt)
@@ -77,6 +87,8 @@ class KVAttention(Part):
         # the framework's grouped attention takes over where nothing here is beyond it
         self.plain = (s.key_dim == s.value_dim and s.chunk is None and not s.out_gate and s.key_dim % 16 == 0
                       and 16 <= s.key_dim <= 256 and self.diff is None and not self.sink and not self.softcap and not self.linear_bias)
+        if self.out_bias:
+            self.kernels = self.kernels + ("sandwich",)
         if self.diff is not None:
             self.kernels = ("gemm", "attention_prep", "attention_diff")
             if rt.dtype == torch.bfloat16 and s.chunk is None:
@@ -109,6 +121,10 @@ class KVAttention(Part):
             p["g"] = ParamSpec((s.num_heads if getattr(s, "gate_per_head", False) else o, H))
         if getattr(s, "value_mix", None) == "mixed":
             p["vmix"] = ParamSpec((), role="vector", init="normal")
+        if getattr(s, "sink_logit", False):
+            p["sink"] = ParamSpec((s.num_heads,), role="vector", init="normal")
+        if getattr(s, "out_bias", False):
+            p["o_bias"] = ParamSpec((H,), role="vector", init="normal")
         if maps == 2:
             p.update({n: ParamSpec((s.key_dim,), role="vector", init="normal") for n in ("lq1", "lk1", "lq2", "lk2")})
         return p
@@ -126,6 +142,8 @@ class KVAttention(Part):
             lq1, lk1, lq2, lk2 = (tensors[n].detach().to("cpu", torch.float64) for n in ("lq1", "lk1", "lq2", "lk2"))
             mixing = torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + float(self.diff)
             self.mixing = mixing.to(torch.float32).reshape(1).to(self.rt.device)
+        self.sink_scores = tensors["sink"].contiguous() if self.sink_logit else None
+        self.o_bias = tensors["o_bias"].contiguous() if self.out_bias else None
         self.v_lambda = tensors["vmix"].reshape(1).contiguous() if "vmix" in tensors else None
 
     def cache_spec(self):
@@ -134,7 +152,7 @@ class KVAttention(Part):
             return PagedKVSpec(s.num_kv_heads, 2 * s.key_dim, s.window, s.value_dim)
         return PagedKVSpec(s.num_kv_heads, s.key_dim, s.window, None if s.value_dim == s.key_dim else s.value_dim)
 
-    def forward(self, x, ctx, cache, writes_cache: bool = True):
+    def forward(self, x, ctx, cache, writes_cache: bool = True, open_sum: bool = False):
         s, ops = self.spec, self.rt.ops
         T = x.shape[0]
         proj = ops.linear(x, self.w_in)                                   # [T, q | k | v | g]
@@ -163,7 +181,13 @@ class KVAttention(Part):
             gate = proj[:, self.q_size + self.k_size + self.v_size:] if s.out_gate else None
             ops.attention_dv(q, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim, ctx, cache, s.scale,
                              s.window or 0, s.chunk or 0, gate, out, **self._softmax_options())
-        return ops.linear(out, self.w_out)
+        y = ops.linear(out, self.w_out)
+        if not self.out_bias:
+            return y
+        if open_sum:
+            return BranchSum([y], [1.0], self.o_bias)
+        ops.branch_sum([y], [1.0], y, bias=self.o_bias)
+        return y
 
     def _prep_options(self, ctx=None) -> dict:
         """Keyword arguments of the preparation kernel that only some specs need."""
@@ -174,6 +198,8 @@ class KVAttention(Part):
             opts["norm_all"] = True
         if self.v_unit:
             opts["v_unit"] = True
+        if self.qk_unit:
+            opts["qk_unit"] = True
         if self.maps > 1:
             opts["maps"] = self.maps
         return opts
@@ -182,6 +208,8 @@ class KVAttention(Part):
         opts = {}
         if self.sink:
             opts["sink"] = True
+        if self.sink_logit:
+            opts["sink_logit"] = self.sink_scores
         if self.gate_per_head and self.spec.out_gate:
             opts["gate_per_head"] = True
         if self.softcap:

@@ -13,6 +13,10 @@ chosen experts; its rows join the 32-bit sum over the chosen experts' rows in th
 with ``shared_gate`` multiplied by the sigmoid of one more 32-bit logit per token, whose row of weights
 stands behind the router's in one matrix.
 
+With ``token_rows`` there is no router: a table of integers, one row per token id, names a token's experts,
+each with the weight 1 / top; the sorting kernel reads it.  A caller that forms the sum over a token's experts
+on its way gets the experts' rows and their places instead (``open_sum``).
+
 The experts' matrices are stacked (``[E, 2F, H]`` with rows alternating gate_i, up_i, and
 ``[E, H, F]``); a step's (token, choice) pairs are sorted by expert on the device into row
 tiles that belong to one expert each, two grouped products run over the used tiles, and the
@@ -26,6 +30,7 @@ from typing import Dict
 import torch
 
 from .base import FEED_FORWARDS, ParamSpec, Part, register_feed_forward
+from .norm import ExpertRows
 
 
 @register_feed_forward("moe")
@@ -51,6 +56,11 @@ class RoutedExperts(Part):
             raise ValueError("a shared expert's gate without a shared expert")
         if getattr(s, "router_bias", False) and getattr(s, "choice_bias", False):
             raise ValueError("a router's bias is part of the logits or for the choice alone, not both")
+        self.token_rows = int(getattr(s, "token_rows", 0))
+        if self.token_rows and (s.weight_on != "output" or self.shared is not None or getattr(s, "router_bias", False)
+                                or getattr(s, "choice_bias", False)):
+            raise ValueError("experts named by a table go with weights on the output, no bias and no shared expert")
+        self.opens_sum = self.token_rows > 0
         if self.shared is not None:
             self.kernels = self.kernels + ("activation",)
 
@@ -60,7 +70,10 @@ class RoutedExperts(Part):
     @classmethod
     def params(cls, spec) -> Dict[str, ParamSpec]:
         H, F = spec.hidden_size, spec.expert_size
-        p = {"router": ParamSpec((spec.num_experts, H))}
+        if getattr(spec, "token_rows", 0):
+            p = {"table": ParamSpec((spec.token_rows, spec.top), role="int_table", init=f"distinct:{spec.num_experts}")}
+        else:
+            p = {"router": ParamSpec((spec.num_experts, H))}
         if getattr(spec, "choice_bias", False):
             p["choice_bias"] = ParamSpec((spec.num_experts,), role="vector", init="normal")
         if getattr(spec, "router_bias", False):
@@ -77,7 +90,13 @@ class RoutedExperts(Part):
     def load(self, tensors):
         s = self.spec
         E, F, H = s.num_experts, s.expert_size, s.hidden_size
-        self.w_router = tensors["router"].contiguous()
+        if self.token_rows:
+            self.table = tensors["table"].contiguous()
+            lo, hi = int(self.table.min()), int(self.table.max())
+            if lo < 0 or hi >= E:
+                raise ValueError(f"the table of experts holds numbers from {lo} to {hi}, there are {E} experts")
+        else:
+            self.w_router = tensors["router"].contiguous()
         if self.shared_gate:                        # the gate's row rides behind the router's
             self.w_router = torch.cat([tensors["router"], tensors["shared_gate"]]).contiguous()
         self.choice_bias = tensors["choice_bias"].contiguous() if "choice_bias" in tensors else None
@@ -88,8 +107,16 @@ class RoutedExperts(Part):
         ).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, open_sum: bool = False):
         s, ops, T = self.spec, self.rt.ops, x.shape[0]
+        if self.token_rows:
+            ids = self.rt.empty(T, s.top, dtype=torch.int32)
+            weights = self.rt.empty(T, s.top, dtype=torch.float32)
+            out = None if open_sum else self.rt.empty(T, s.hidden_size)
+            extra = {"limit": float(s.limit)} if s.limit else {}
+            got = ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, s.activation, s.weight_on, out, gated=self.gated,
+                                  by_token=(self.table, ctx.token_ids), open_sum=open_sum, **extra)
+            return ExpertRows(got[0], got[1], weights) if open_sum else out
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
         out = self.rt.empty(T, s.hidden_size)
         extra = {}

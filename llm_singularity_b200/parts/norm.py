@@ -26,6 +26,26 @@ class NormedDelta:
         self.values, self.weight, self.eps, self.mult = values, weight, float(eps), float(mult)
 
 
+class BranchSum:
+    """A sublayer's result that is still the sum of several: ``sum_b scales[b] * values[b] + bias`` (``bias``
+    32-bit or None).  Handed on where the kernel that takes it forms the sum itself."""
+
+    __slots__ = ("values", "scales", "bias")
+
+    def __init__(self, values, scales, bias=None):
+        self.values, self.scales, self.bias = list(values), [float(s) for s in scales], bias
+
+
+class ExpertRows:
+    """A routed feed-forward's result before the sum over a token's experts: ``sum_k weights[t, k] *
+    rows[places[t * top + k]]``."""
+
+    __slots__ = ("rows", "places", "weights")
+
+    def __init__(self, rows: torch.Tensor, places: torch.Tensor, weights: torch.Tensor):
+        self.rows, self.places, self.weights = rows, places, weights
+
+
 class DeltaPair:
     """Two sublayers' outputs that both still have to join the stream (sublayers that read one input side by
     side).  Handed on in place of a plain delta: the norm that takes it adds both in 32-bit."""
@@ -78,6 +98,20 @@ class RMSNorm(Part):
         out = self.rt.empty(n, residual.shape[1])
         self.rt.ops.stream_norm(residual, y, w, eps, mult, step, rows, self.weight, self.spec.eps, out)
         return out
+
+    def join(self, residual: torch.Tensor, delta) -> torch.Tensor:
+        """residual += norm(delta) in place (this norm stands behind the sublayer that made ``delta``: a tensor,
+        a ``BranchSum`` or ``ExpertRows``); returns the stream as a product's operand (a rounded copy, or
+        the stream itself in 32-bit)."""
+        copy = None if self.rt.dtype == torch.float32 else self.rt.empty(*residual.shape)
+        if isinstance(delta, ExpertRows):
+            self.rt.ops.join_norm(residual, [delta.rows], [1.0], None, self.weight, self.spec.eps, copy, pos=delta.places,
+                                  wts=delta.weights)
+        elif isinstance(delta, BranchSum):
+            self.rt.ops.join_norm(residual, delta.values, delta.scales, delta.bias, self.weight, self.spec.eps, copy)
+        else:
+            self.rt.ops.join_norm(residual, [delta], [1.0], None, self.weight, self.spec.eps, copy)
+        return residual if copy is None else copy
 
     def fold(self):
         """What a product needs to take this norm upon itself: the weight and eps."""

@@ -8,8 +8,10 @@ The spec's ``gate`` says where a and b come from: one constant per head and a ke
 ("fixed_decay": S decays uniformly, b = act(W_k x)), or a forget gate per channel with a learnt
 floor that also sets the write strength ("forget": a = floor + (1 - floor) sigmoid(W_f x + bias),
 b = 1 - a; no key, no other scale).  The outputs are RMS-normed (all heads together with one weight
-over the row, or each head by itself with one weight of head size), optionally multiplied by
-sigmoid(W_g x), and projected by W_o.
+over the row, or each head by itself with one weight of head size or none), optionally multiplied by
+sigmoid or silu of W_g x, and projected by W_o.  With a fixed decay q and k may be rotated by the tokens'
+positions and k scaled (retention); the projections then leave their product in 32-bit and are rotated
+there, so that nothing that enters the recurrence is rounded behind its projection.
 
 The state starts at zero when a request takes a slot, is 32-bit, and is carried from step to
 step in the slot's row of a ``StateSpec`` cache.  One product makes all projections of a step
@@ -23,7 +25,7 @@ from typing import Dict
 
 import torch
 
-from .base import ParamSpec, Part, StateSpec, register_mixer
+from .base import POSITIONS, ParamSpec, Part, StateSpec, register_mixer
 
 
 @register_mixer("linear_recurrence")
@@ -38,8 +40,24 @@ class LinearRecurrence(Part):
             raise ValueError(f"gate '{s.gate}' is not known (fixed_decay, forget)")
         if s.gate == "fixed_decay" and len(s.decay) != s.num_heads:
             raise ValueError(f"{len(s.decay)} decays for {s.num_heads} heads")
-        if s.out_norm not in ("all", "per_head"):
-            raise ValueError(f"out_norm '{s.out_norm}' is not known (all, per_head)")
+        if s.out_norm not in ("all", "per_head", "unit"):
+            raise ValueError(f"out_norm '{s.out_norm}' is not known (all, per_head, unit)")
+        self.gate_act = getattr(s, "out_gate_activation", "sigmoid")
+        if self.gate_act not in ("sigmoid", "silu"):
+            raise ValueError(f"out_gate_activation '{self.gate_act}' is not known (sigmoid, silu)")
+        position = getattr(s, "position", None)
+        self.position = POSITIONS.build(position, rt) if position is not None and position.kind != "none" else None
+        self.table = self.position.rotary_table() if self.position is not None else None
+        if self.position is not None and (self.table is None or getattr(position, "pairing", "half") != "half"
+                                          or s.gate != "fixed_decay" or s.q_activation != "none" or s.k_activation != "none"):
+            raise ValueError("a rotation of q and k is in halves and goes with a fixed decay, without activations on q and k")
+        self.k_scale = float(getattr(s, "k_scale", 1.0))
+        if self.k_scale != 1.0 and s.gate != "fixed_decay":
+            raise ValueError("a factor on k goes with a fixed decay")
+        # the output kernel that knows heads without a weight and the silu gate
+        self.plain_output = s.out_norm != "unit" and self.gate_act == "sigmoid"
+        if not self.plain_output:
+            self.kernels = self.kernels + ("delta_rule",)
         for a in (s.q_activation, s.k_activation, s.v_activation):
             if a not in ("none", "silu"):
                 raise ValueError(f"activation '{a}' is not implemented here (none, silu)")
@@ -62,6 +80,8 @@ class LinearRecurrence(Part):
             p["floor"] = ParamSpec((qk,), role="vector", init="normal")
         if spec.out_gate:
             p["g"] = ParamSpec((vv, H))
+        if spec.out_norm == "unit":
+            return p
         p["norm"] = ParamSpec((vv if spec.out_norm == "all" else spec.value_dim,), role="vector", init="ones")
         return p
 
@@ -71,7 +91,7 @@ class LinearRecurrence(Part):
         rows = [tensors["q"], second, tensors["v"]] + ([tensors["g"]] if s.out_gate else [])
         self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_out = tensors["o"].contiguous()
-        self.norm = tensors["norm"]
+        self.norm = tensors.get("norm")
         self.f_bias = tensors.get("f_bias")
         self.floor = tensors.get("floor")
 
@@ -81,12 +101,21 @@ class LinearRecurrence(Part):
 
     def forward(self, x, ctx, cache, writes_cache: bool = True):
         s, ops = self.spec, self.rt.ops
-        proj = ops.linear(x, self.w_in)                               # [T, q | k or f | v | g]
+        # [T, q | k or f | v | g]
+        proj = ops.linear(x, self.w_in) if self.position is None else ops.linear(x, self.w_in, out_dtype=torch.float32)
+        if self.position is not None:
+            ops.turn_heads(proj, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx)
         o = self.rt.empty(x.shape[0], self.vv, dtype=torch.float32)
+        # (a factor on k is one on the read-out: it rides on q)
+        extra = {"q_scale": self.k_scale} if self.k_scale != 1.0 else {}
         ops.linear_scan(proj, 0, self.qk, 2 * self.qk, s.num_heads, s.key_dim, s.value_dim, s.gate,
                         self.decay, self.f_bias, self.floor, s.q_activation, s.k_activation, s.v_activation,
-                        cache.state, ctx, o)
+                        cache.state, ctx, o, **extra)
         gate = proj[:, 2 * self.qk + self.vv:] if s.out_gate else None
         y = self.rt.empty(x.shape[0], self.vv)
-        ops.rows_norm_gate(o, self.norm, 1 if s.out_norm == "all" else s.num_heads, s.eps, gate, y)
+        heads = 1 if s.out_norm == "all" else s.num_heads
+        if self.plain_output:
+            ops.rows_norm_gate(o, self.norm, heads, s.eps, gate, y)
+        else:
+            ops.delta_output(o, self.norm, heads, s.eps, gate, self.gate_act if gate is not None else "none", y)
         return ops.linear(y, self.w_out)

@@ -115,6 +115,8 @@ def _register_builtin() -> None:
     register_architecture(ZinizenConfig.architecture, ZinizenConfig)
     from .config.mofidra import MofidraConfig
     register_architecture(MofidraConfig.architecture, MofidraConfig)
+    from .config.lilupel import LilupelConfig
+    register_architecture(LilupelConfig.architecture, LilupelConfig)
 
 
 _register_builtin()

@@ -22,6 +22,7 @@ that IEEE 754 pins down, which library functions are not.
 from __future__ import annotations
 
 import json
+import math
 import os
 import zlib
 from typing import Dict, Mapping, Tuple
@@ -115,18 +116,37 @@ def normal_tensor(shape, key: int, mean: float, scale: float, dtype: torch.dtype
     return out.reshape(tuple(shape))
 
 
+def distinct_rows(shape, key: int, n: int) -> torch.Tensor:
+    """int32 [rows, cols] whose rows hold different numbers below ``n``: a start and a step per row from the
+    counter-based stream, the step prime to ``n``."""
+    rows, cols = shape
+    if cols > n:
+        raise ValueError(f"rows of {cols} different numbers below {n}")
+    steps = np.array([x for x in range(1, n + 1) if math.gcd(x, n) == 1], dtype=np.int64)
+    with np.errstate(over="ignore"):
+        z = np.uint64(key) + np.arange(1, rows + 1, dtype=np.uint64) * np.uint64(_GOLDEN)
+        z = (z ^ (z >> np.uint64(30))) * np.uint64(0xBF58476D1CE4E5B9)
+        z = (z ^ (z >> np.uint64(27))) * np.uint64(0x94D049BB133111EB)
+        z = z ^ (z >> np.uint64(31))
+    start = ((z >> np.uint64(40)).astype(np.int64) % n)[:, None]
+    step = steps[(z & np.uint64(0xFFFFFF)).astype(np.int64) % len(steps)][:, None]
+    return torch.from_numpy(((start + np.arange(cols, dtype=np.int64)[None, :] * step) % n).astype(np.int32))
+
+
 def random_tensors(expected: Mapping[str, Tuple[Tuple[int, ...], str, str]], seed: int,
                    dtype: torch.dtype = torch.bfloat16, std: float = 0.02,
                    norm_noise: float = 0.0, device="cpu") -> Dict[str, torch.Tensor]:
     """``expected``: name -> (shape, role, init).  Matrices/tables in ``dtype``, vectors in
-    ``dtype`` too (a checkpoint stores one dtype), integer tables as int32 zeros.  The same
+    ``dtype`` too (a checkpoint stores one dtype), integer tables as int32 (zeros, or
+    rows of different numbers where ``init`` asks for them).  The same
     values whatever ``device`` is."""
     out: Dict[str, torch.Tensor] = {}
     for name, (shape, role, init) in expected.items():
-        if role == "int_table":
-            out[name] = torch.zeros(shape, dtype=torch.int32, device=device)
-            continue
         key = tensor_key(seed, name)
+        if role == "int_table":
+            out[name] = (distinct_rows(shape, key, int(init.split(":")[1])) if init.startswith("distinct:")
+                         else torch.zeros(shape, dtype=torch.int32)).to(device)
+            continue
         if init == "ones":
             out[name] = normal_tensor(shape, key, 1.0, norm_noise, dtype, device)
         else:
