@@ -321,6 +321,104 @@ linear_scan_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
     }
 }
 
+// A step that brings every request one token: no walk, the state is read, updated and written once and that
+// is all there is.  A block has `kSingleRows` value columns of a (request, head); LANES lanes hold a column's key
+// channels as 16-byte vectors (key_dim a multiple of four), a column's rows in flight together.  The state
+// is asked for (L2) before the kernel in front has ended.
+constexpr int kSingleRows = 32;
+
+template <typename T>
+__device__ __forceinline__ void single_gates(float& a, float& b, float z, int gate, float fixed, float keep, float write, int k_act,
+                                             const float* floor_, const float* f_bias, int c) {
+    if (gate == 1) {
+        const float lo = floor_[c];
+        a = lo + (1.f - lo) * scan_sigmoid<T>(z + (f_bias ? f_bias[c] : 0.f));
+        b = 1.f - a;
+    } else {
+        a = gate == 0 ? fixed : keep;
+        b = (gate == 0 ? 1.f : write) * scan_act<T>(z, k_act);
+    }
+}
+
+template <typename T, int LANES>
+__global__ void __launch_bounds__(kScanThreads)
+single_token_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_off, int v_off, int heads, int D, int V, int gate,
+                    const float* __restrict__ decay, const float* __restrict__ f_bias, const float* __restrict__ floor_, int q_act,
+                    int k_act, int v_act, float* __restrict__ state, int n_slots, const int* __restrict__ q_start,
+                    const int* __restrict__ table_rows, float* __restrict__ out, const float* __restrict__ g_keep,
+                    const float* __restrict__ g_write, int ones, float q_scale, int share) {
+    extern __shared__ float4 sh4[];
+    float* q_sh = reinterpret_cast<float*>(sh4);             // D
+    float* a_sh = q_sh + D;
+    float* b_sh = a_sh + D;
+    float* v_sh = b_sh + D;                                  // kSingleRows
+    lsb_pdl_launch_dependents();
+    const int r = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * kSingleRows, Vs = V + ones;
+    const int t = q_start[r], slot = table_rows[r];
+    const int cols = min(kSingleRows, Vs - col0);
+    if (slot < 0 || slot >= n_slots) {
+        if (threadIdx.x == 0) lsb_set_status(LSB_BAD_ROW);
+        return;
+    }
+    float* base = state + (((size_t)slot * heads + h) * Vs + col0) * D;
+    for (int i = threadIdx.x * 32; i < cols * D; i += kScanThreads * 32)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(base + i));
+    lsb_pdl_wait();
+    const T* row = proj + (size_t)t * ld;
+    const int hD = h / share * D;
+    const float fixed = gate == 0 ? decay[h] : 0.f;
+    const float keep = gate == 2 ? g_keep[(size_t)t * heads + h] : 0.f, write = gate == 2 ? g_write[(size_t)t * heads + h] : 0.f;
+    for (int d = threadIdx.x; d < D; d += kScanThreads) {
+        q_sh[d] = scan_act<T>(lsb_to_float(row[q_off + hD + d]), q_act) * q_scale;
+        single_gates<T>(a_sh[d], b_sh[d], lsb_to_float(row[k_off + hD + d]), gate, fixed, keep, write, k_act, floor_, f_bias, h * D + d);
+    }
+    for (int c = threadIdx.x; c < cols; c += kScanThreads)
+        v_sh[c] = col0 + c < V ? scan_act<T>(lsb_to_float(row[v_off + h * V + col0 + c]), v_act) : 1.f;
+    __syncthreads();
+    constexpr int PER_WARP = 32 / LANES;                    // columns a warp has at a time
+    constexpr int STRIDE = PER_WARP * (kScanThreads / 32), AHEAD = 8;
+    const int lane = threadIdx.x & 31, part = lane % LANES, first = (threadIdx.x >> 5) * PER_WARP + lane / LANES;
+    const int vecs = D >> 2;
+    for (int c0 = first; c0 - lane / LANES < cols; c0 += STRIDE * AHEAD) {     // (a warp's lanes leave together)
+        float acc[AHEAD];
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) acc[k] = 0.f;
+        for (int x = part; x - part < vecs; x += LANES) {
+            const bool in = x < vecs;
+            float4 s[AHEAD];
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) {
+                const int c = c0 + k * STRIDE;
+                s[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (in && c < cols) s[k] = *reinterpret_cast<const float4*>(base + (size_t)c * D + 4 * x);
+            }
+            if (!in) continue;
+            const float4 q = *reinterpret_cast<const float4*>(q_sh + 4 * x), a = *reinterpret_cast<const float4*>(a_sh + 4 * x),
+                         b = *reinterpret_cast<const float4*>(b_sh + 4 * x);
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) {
+                const int c = c0 + k * STRIDE;
+                if (c < cols) {
+                    const float v = v_sh[c];
+                    s[k].x = a.x * s[k].x + b.x * v;
+                    s[k].y = a.y * s[k].y + b.y * v;
+                    s[k].z = a.z * s[k].z + b.z * v;
+                    s[k].w = a.w * s[k].w + b.w * v;
+                    *reinterpret_cast<float4*>(base + (size_t)c * D + 4 * x) = s[k];
+                    acc[k] += s[k].x * q.x + s[k].y * q.y + s[k].z * q.z + s[k].w * q.w;
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+#pragma unroll
+            for (int o = LANES >> 1; o > 0; o >>= 1) acc[k] += __shfl_xor_sync(0xffffffffu, acc[k], o);
+            const int c = c0 + k * STRIDE;
+            if (part == 0 && c < cols) out[(size_t)t * heads * Vs + (size_t)h * Vs + col0 + c] = acc[k];
+        }
+    }
+}
+
 // start(0) = the slot's state; start(s + 1) = P_s * start(s) + E_s.  seg_state holds E_s coming in
 // and start(s) going out; the slot gets the state after the last segment.
 __global__ void scan_chain_kernel(float* __restrict__ state, int n_slots, float* __restrict__ seg_state,
@@ -389,6 +487,20 @@ LSB_API int lsb_linear_scan(const void* proj, int dtype, long long ld, int q_off
         return (int)cudaErrorInvalidValue;
     ones = ones ? 1 : 0;
     const int Vs = V + ones;
+    if (max_q_len == 1 && D % 4 == 0 && (uintptr_t)state % 16 == 0) {        // single tokens only
+        const dim3 grid((Vs + kSingleRows - 1) / kSingleRows, heads, n_requests);
+        const size_t smem = (size_t)(3 * D + kSingleRows) * sizeof(float);
+#define LSB_SINGLE(LANES)                                                                                            \
+    LSB_DISPATCH_DTYPE(dtype, return lsb_launch(single_token_kernel<T, LANES>, grid, dim3(kScanThreads), smem, stream, 1, \
+                                                (const T*)proj, ld, q_off, k_off, v_off, heads, D, V, gate, decay, f_bias, \
+                                                floor_, q_act, k_act, v_act, state, n_slots, q_start, table_rows, out, g_keep, \
+                                                g_write, ones, q_scale, heads / key_heads))
+        if (D > 64) LSB_SINGLE(32);
+        else if (D > 32) LSB_SINGLE(16);
+        else if (D > 16) LSB_SINGLE(8);
+        else LSB_SINGLE(4);
+#undef LSB_SINGLE
+    }
     int split, per;
     scan_shape(D, &split, &per);
     const int cols = kScanThreads / split;

@@ -1009,7 +1009,8 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
                 value_dim: int, gate: str, decay: Optional[torch.Tensor], f_bias: Optional[torch.Tensor],
                 floor: Optional[torch.Tensor], q_act: str, k_act: str, v_act: str, state: torch.Tensor,
                 ctx, out: torch.Tensor, keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
-                ones: bool = False, q_scale: float = 1.0, key_heads: Optional[int] = None) -> None:
+                ones: bool = False, q_scale: float = 1.0, key_heads: Optional[int] = None,
+                requests: Optional[int] = None) -> None:
     """S <- diag(a) S + b v^T, o = S^T q per head and token, each request from its slot's state
     (``state`` [slots, heads, value_dim, key_dim] 32-bit, updated in place); ``proj`` [T, columns] holds
     the projections of q at ``q_off``, of k (or the forget gate) at ``k_off`` and of v at ``v_off``;
@@ -1019,7 +1020,8 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     of a head.  ``ones``: a value column of ones rides along behind each head's ``value_dim`` columns
     (state and out then have ``value_dim + 1`` columns a head, the last one of out being the
     running sum of b dotted with q).  ``q_scale`` multiplies q.  ``key_heads``: heads of q and k, shared by
-    groups of ``heads / key_heads`` heads (not with the forget gate)."""
+    groups of ``heads / key_heads`` heads (not with the forget gate).  ``requests``: only the step's first that
+    many, which bring one token each."""
     _req(proj, "proj", dim=2)
     _req(state, "state", torch.float32, 4)
     _req(out, "out", torch.float32, 2)
@@ -1049,7 +1051,8 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     # a few requests with long portions: segments walked side by side (twice the arithmetic, a chain
     # a segment long); many requests, short portions and single tokens: one walk each
     seg, seg_state, seg_decay = 0, None, None
-    if SCAN_SEGMENT and ctx.max_q_len >= 2 * SCAN_SEGMENT and ctx.n_requests <= 8:
+    n_req, max_q = (ctx.n_requests, ctx.max_q_len) if requests is None else (requests, 1)
+    if SCAN_SEGMENT and max_q >= 2 * SCAN_SEGMENT and n_req <= 8:
         seg = SCAN_SEGMENT
         n = ctx.n_requests * -(-ctx.max_q_len // seg)
         seg_state = torch.empty(n * heads * cols * key_dim, dtype=torch.float32, device=proj.device)
@@ -1057,15 +1060,16 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     _call("linear_scan", "lsb_linear_scan", _p(proj), _i(_dt(proj)), _ll(ld), _i(q_off), _i(k_off), _i(v_off),
           _i(heads), _i(key_dim), _i(value_dim), _i(SCAN_GATES[gate]), _p(decay), _p(f_bias), _p(floor),
           _i(_SCAN_ACTS[q_act]), _i(_SCAN_ACTS[k_act]), _i(_SCAN_ACTS[v_act]), _p(state), _i(state.shape[0]),
-          _p(ctx.q_start), _p(ctx.table_rows), _i(ctx.n_requests), _p(out), _i(seg), _i(ctx.max_q_len),
+          _p(ctx.q_start), _p(ctx.table_rows), _i(n_req), _p(out), _i(seg), _i(max_q),
           _p(seg_state), _p(seg_decay), _p(keep), _p(write), _i(1 if ones else 0), _f(q_scale), _i(key_heads),
           _stream(out))
 
 
-def turn_heads(proj: torch.Tensor, q_off: int, k_off: int, heads: int, key_dim: int, inv_freq: torch.Tensor, ctx) -> None:
+def turn_heads(proj: torch.Tensor, q_off: int, k_off: int, heads: int, key_dim: int, inv_freq: torch.Tensor, ctx,
+               tokens: Optional[int] = None) -> None:
     """The first ``2 * len(inv_freq)`` channels of every head of q and k (``heads`` heads of ``key_dim`` from
     ``q_off`` and ``k_off`` on in the 32-bit rows of ``proj``) turned by the token's position, in place: pairs
-    (i, i + half) by ``pos * inv_freq[i]``."""
+    (i, i + half) by ``pos * inv_freq[i]``.  ``tokens``: only the step's first that many."""
     _req(proj, "proj", torch.float32, 2)
     _req(inv_freq, "inv_freq", torch.float32, 1)
     T, ld = proj.shape
@@ -1073,7 +1077,85 @@ def turn_heads(proj: torch.Tensor, q_off: int, k_off: int, heads: int, key_dim: 
     if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off) < 0 or max(q_off, k_off) + heads * key_dim > ld:
         raise KernelError("turn_heads: proj, the heads and the step disagree")
     _call("linear_scan", "lsb_turn_heads", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(heads), _i(key_dim), _i(dims),
-          _p(inv_freq), _p(ctx.positions), _i(T), _stream(proj))
+          _p(inv_freq), _p(ctx.positions), _i(T if tokens is None else tokens), _stream(proj))
+
+
+# ---------------------------------------- memories that fade by one number per head: prompts on the tensor cores
+CHUNK_SCAN = True               # bfloat16 portions of at least CHUNK_SCAN_FROM tokens (csrc/chunk_scan.cu)
+CHUNK_SCAN_FROM = 48
+
+
+def chunk_scan_first(ctx, dtype, key_dim: int, value_dim: int) -> Optional[int]:
+    """The first request of the step that the chunked form takes (with all after it; the ones before bring one
+    token each and are walked), or None if the whole step is walked."""
+    if not CHUNK_SCAN or dtype != torch.bfloat16 or ctx.max_q_len < CHUNK_SCAN_FROM \
+            or not _lib("chunk_scan").lsb_chunk_scan_supported(_i(key_dim), _i(value_dim)):
+        return None
+    n_decode, first, last = _batch_shape(ctx)
+    return first if n_decode == first and last == ctx.n_requests else 0
+
+
+def turn_split(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, key_dim: int, value_dim: int,
+               inv_freq: torch.Tensor, ctx, first: int) -> torch.Tensor:
+    """Rows for ``chunk_scan`` from the 32-bit rows of ``proj``: q and k turned as ``turn_heads`` does, each as a
+    rounded value and a rounded rest, and v rounded: bfloat16 [T, q | rest | k | rest | v], filled from the token
+    ``first`` on."""
+    _req(proj, "proj", torch.float32, 2)
+    _req(inv_freq, "inv_freq", torch.float32, 1)
+    T, ld = proj.shape
+    qk, vv, dims = heads * key_dim, heads * value_dim, 2 * inv_freq.shape[0]
+    if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off, v_off) < 0 or max(q_off, k_off) + qk > ld or v_off + vv > ld:
+        raise KernelError("turn_split: proj, the heads and the step disagree")
+    rows = torch.empty(T, 4 * qk + vv, dtype=torch.bfloat16, device=proj.device)
+    _call("chunk_scan", "lsb_turn_split", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(heads), _i(key_dim), _i(vv), _i(dims),
+          _p(inv_freq), _p(ctx.positions), _i(first), _i(T - first), _p(rows), _stream(proj))
+    return rows
+
+
+def _chunk_scratch(name: str, numel: int, device, dtype) -> torch.Tensor:
+    """A scratch buffer of at least ``numel`` elements, kept for reuse (the largest asked for so far)."""
+    key = ("chunk_scan", name, device)
+    got = _scratch.get(key)
+    if got is None or got.numel() < numel:
+        if torch.cuda.is_current_stream_capturing():
+            return torch.empty(numel, dtype=dtype, device=device)
+        got = _scratch[key] = torch.empty(numel, dtype=dtype, device=device)
+    return got
+
+
+def chunk_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, key_heads: int, key_dim: int, value_dim: int,
+               state: torch.Tensor, ctx, out: torch.Tensor, first: int, *, q_lo: int = -1, k_lo: int = -1,
+               log_keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
+               log_decay: Optional[torch.Tensor] = None, q_scale: float = 1.0) -> None:
+    """What ``linear_scan`` does for a memory that fades by one number per head and token, for the requests from
+    ``first`` on, in chunks on the tensor cores.  ``rows`` bfloat16: q, k and v at their offsets, with ``q_lo`` / ``k_lo``
+    the rounded rests of q and k.  ``log_keep`` and ``write`` (32-bit [T, heads]): the logarithm of the fade and the
+    factor of a write; or ``log_decay`` [heads], the same for every token, with writes as they are."""
+    _req(rows, "rows", torch.bfloat16, 2)
+    _req(state, "state", torch.float32, 4)
+    _req(out, "out", torch.float32, 2)
+    T, ld = rows.shape
+    if state.shape[1:] != (heads, value_dim, key_dim) or out.shape != (T, heads * value_dim) or ctx.n_tokens != T:
+        raise KernelError("chunk_scan: state, out or the step do not fit the sizes")
+    for off, n in ((q_off, key_heads * key_dim), (k_off, key_heads * key_dim), (v_off, heads * value_dim)) + \
+            (((q_lo, key_heads * key_dim), (k_lo, key_heads * key_dim)) if q_lo >= 0 else ()):
+        if off < 0 or off + n > ld:
+            raise KernelError("chunk_scan: an operand lies outside the rows")
+    for name, t, shape in (("log_keep", log_keep, (T, heads)), ("write", write, (T, heads)), ("log_decay", log_decay, (heads,))):
+        if t is not None:
+            _req(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"chunk_scan: {name} must be {list(shape)}")
+    n_req = ctx.n_requests - first
+    n = T // int(_lib("chunk_scan").lsb_chunk_tokens()) + n_req
+    gain = _chunk_scratch("gain", n * heads * value_dim * key_dim, rows.device, torch.float32)
+    starts = _chunk_scratch("starts", n * heads * 2 * value_dim * key_dim, rows.device, torch.bfloat16)
+    fade = _chunk_scratch("fade", n * heads, rows.device, torch.float32)
+    _call("chunk_scan", "lsb_chunk_scan", _p(rows), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(q_lo), _i(k_lo), _i(heads),
+          _i(key_heads), _i(key_dim), _i(value_dim), _p(log_keep), _p(write), _p(log_decay), _f(q_scale), _p(state),
+          _i(state.shape[0]), ctypes.c_void_p(ctx.q_start.data_ptr() + 4 * first),
+          ctypes.c_void_p(ctx.table_rows.data_ptr() + 4 * first), _i(n_req), _i(ctx.max_q_len), _p(out), _p(gain), _p(starts),
+          _p(fade), _stream(out))
 
 
 # ----------------------------------------------------------------- state-space memory

@@ -48,6 +48,7 @@ SOURCES: Dict[str, object] = {          # library -> its source file (or files)
     "sandwich": "sandwich.cu",
     "output_norm": "output_norm.cu",
     "state_space": "state_space.cu",
+    "chunk_scan": "chunk_scan.cu",
     "attention_prep": "attention_prep.cu",
     "attention_dv": "attention_dv.cu",
     "attention_diff": "attention_diff.cu",

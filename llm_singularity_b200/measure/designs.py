@@ -1,4 +1,11 @@
-"""Prefill and decode throughput of a design (Ridotar, Fogezen, Fikizen, Zinizen, Mofidra) beside the Llama decoder at equal size.
+"""Prefill and decode throughput of a design (Ridotar, Fogezen, Fikizen, Zinizen, Mofidra, Lilupel) beside the Llama decoder at equal size.
+
+Lilupel: layers cycling through the parallel pair (windowed sink attention with normed heads beside a
+retention memory), two state-space memories (twice the width inside, heads of 64, 128 state channels, one
+group, four taps) and the first layer's weights once more; every layer's feed-forward sends a token to the
+``top`` experts that a table names.  It is also run beside Ridotar (linear recurrences, routed
+experts) and Fikizen (windowed sink attention, a parallel pair, memories behind short convolutions),
+the designs closest to it.
 
 Mofidra: differential attention (two maps of 64 over values of 128 per head, as many heads and kv heads
 as the Llama model) beside the feed-forward in every layer; the first layer's feed-forward is dense,
@@ -143,10 +150,29 @@ def mofidra_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:
             "loop": {"start": 1, "stop": 2, "times": 2 if layers > 2 else 1}}
 
 
+def lilupel_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:
+    heads = width // 128
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    pair = {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                     "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": 128}},
+            "right": {"heads": heads, "dim": 64, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 5 * h / heads) for h in range(heads)],
+                      "rot": {"base": 10000.0, "dims": 64}},
+            "left_scale": 0.6, "right_scale": 0.9}
+    space = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    out = []
+    for i in range(layers):
+        e = {"type": "mamba2" if i % 4 in (1, 2) else "parallel", "mlp": mlp}
+        e["mixer"] = dict(space) if e["type"] == "mamba2" else dict(pair)
+        if i % 4 == 3:
+            e["weights_of"] = 0
+        out.append(e)
+    return {"architecture": "Lilupel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": out}
+
+
 DESIGNS = {"ridotar": ridotar_config, "fogezen": fogezen_config, "fikizen": fikizen_config, "zinizen": zinizen_config,
-           "mofidra": mofidra_config}
+           "mofidra": mofidra_config, "lilupel": lilupel_config}
 # the designs each is also measured beside (Llama always is)
-CLOSEST = {"fikizen": ("fogezen",), "zinizen": ("ridotar",), "mofidra": ("zinizen",)}
+CLOSEST = {"fikizen": ("fogezen",), "zinizen": ("ridotar",), "mofidra": ("zinizen",), "lilupel": ("ridotar", "fikizen")}
 
 
 def llama_config(width, layers, experts, top, ff, kv_rank, vocab) -> dict:

@@ -54,6 +54,8 @@ class LinearRecurrence(Part):
         self.k_scale = float(getattr(s, "k_scale", 1.0))
         if self.k_scale != 1.0 and s.gate != "fixed_decay":
             raise ValueError("a factor on k goes with a fixed decay")
+        if self.position is not None and rt.dtype == torch.bfloat16:
+            self.kernels = self.kernels + ("chunk_scan",)
         # the output kernel that knows heads without a weight and the silu gate
         self.plain_output = s.out_norm != "unit" and self.gate_act == "sigmoid"
         if not self.plain_output:
@@ -63,9 +65,12 @@ class LinearRecurrence(Part):
                 raise ValueError(f"activation '{a}' is not implemented here (none, silu)")
         self.qk = s.num_heads * s.key_dim
         self.vv = s.num_heads * s.value_dim
-        self.decay = None
+        self.decay = self.log_decay = None
         if s.gate == "fixed_decay":
-            self.decay = torch.tensor([float(d) for d in s.decay], dtype=torch.float32, device=rt.device)
+            decay = torch.tensor([float(d) for d in s.decay], dtype=torch.float64)
+            self.decay = decay.to(dtype=torch.float32, device=rt.device)
+            if bool((decay >= 0).all()):
+                self.log_decay = torch.log(decay).to(dtype=torch.float32, device=rt.device)
 
     @classmethod
     def params(cls, spec) -> Dict[str, ParamSpec]:
@@ -99,18 +104,34 @@ class LinearRecurrence(Part):
         s = self.spec
         return StateSpec((s.num_heads, s.value_dim, s.key_dim))     # key channels contiguous
 
+    def _walk(self, proj, ctx, cache, o, **extra):
+        s = self.spec
+        if self.k_scale != 1.0:                     # (a factor on k is one on the read-out: it rides on q)
+            extra["q_scale"] = self.k_scale
+        self.rt.ops.linear_scan(proj, 0, self.qk, 2 * self.qk, s.num_heads, s.key_dim, s.value_dim, s.gate,
+                                self.decay, self.f_bias, self.floor, s.q_activation, s.k_activation, s.v_activation,
+                                cache.state, ctx, o, **extra)
+
     def forward(self, x, ctx, cache, writes_cache: bool = True):
         s, ops = self.spec, self.rt.ops
         # [T, q | k or f | v | g]
         proj = ops.linear(x, self.w_in) if self.position is None else ops.linear(x, self.w_in, out_dtype=torch.float32)
-        if self.position is not None:
-            ops.turn_heads(proj, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx)
         o = self.rt.empty(x.shape[0], self.vv, dtype=torch.float32)
-        # (a factor on k is one on the read-out: it rides on q)
-        extra = {"q_scale": self.k_scale} if self.k_scale != 1.0 else {}
-        ops.linear_scan(proj, 0, self.qk, 2 * self.qk, s.num_heads, s.key_dim, s.value_dim, s.gate,
-                        self.decay, self.f_bias, self.floor, s.q_activation, s.k_activation, s.v_activation,
-                        cache.state, ctx, o, **extra)
+        if self.position is None:
+            self._walk(proj, ctx, cache, o)
+        else:
+            # prompt portions in chunks on the tensor cores where they can be, the rest walked
+            first = ops.chunk_scan_first(ctx, self.rt.dtype, s.key_dim, s.value_dim) if self.log_decay is not None else None
+            walked = ctx.n_requests if first is None else first
+            if walked:
+                tokens = {} if first is None else {"tokens": first}
+                ops.turn_heads(proj, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx, **tokens)
+                self._walk(proj, ctx, cache, o, **({} if first is None else {"requests": first}))
+            if first is not None:
+                qk = self.qk
+                rows = ops.turn_split(proj, 0, qk, 2 * qk, s.num_heads, s.key_dim, s.value_dim, self.table[0], ctx, first)
+                ops.chunk_scan(rows, 0, 2 * qk, 4 * qk, s.num_heads, s.num_heads, s.key_dim, s.value_dim, cache.state, ctx, o,
+                               first, q_lo=qk, k_lo=3 * qk, log_decay=self.log_decay, q_scale=self.k_scale)
         gate = proj[:, 2 * self.qk + self.vv:] if s.out_gate else None
         y = self.rt.empty(x.shape[0], self.vv)
         heads = 1 if s.out_norm == "all" else s.num_heads

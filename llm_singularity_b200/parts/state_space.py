@@ -10,7 +10,8 @@ x, B and C pass a short causal convolution over time per channel, with a bias, a
 y times silu(z) is RMS-normed in ``norm_groups`` equal parts with one weight over the row, and projected.
 
 The walk is the one of linear attention (``csrc/linear_scan.cu``) with C for the query, B for the key, x for the
-value and two numbers per token and head given from outside, exp(-exp(A_log) dt) and dt.  The projection leaves
+value and two numbers per token and head given from outside, exp(-exp(A_log) dt) and dt; prompt portions run
+in chunks on the tensor cores where the sizes allow (``csrc/chunk_scan.cu``).  The projection leaves
 its product in 32-bit; a kernel in front of the walk convolves and makes the two numbers, a kernel
 behind it adds D x, gates and norms.  The state S and the convolution's last ``conv_taps - 1`` inputs are
 32-bit ``StateSpec`` rows, zero when a request takes a slot.
@@ -40,6 +41,9 @@ class StateSpace(Part):
         if s.norm_groups < 1 or self.inner % s.norm_groups:
             raise ValueError(f"{s.norm_groups} norm groups do not divide a row of {self.inner}")
         self.channels = self.inner + 2 * self.gn
+        self.aligned = s.value_dim % 8 == 0 and s.state_dim % 8 == 0         # (16-byte rows of every operand)
+        if self.aligned and rt.dtype == torch.bfloat16:
+            self.kernels = self.kernels + ("chunk_scan",)
 
     @classmethod
     def params(cls, spec) -> Dict[str, ParamSpec]:
@@ -77,8 +81,14 @@ class StateSpace(Part):
         ops.state_space_prep(proj, x_off, dt_off, self.channels, self.conv, self.conv_bias, self.dt_bias, self.a_log, conv_state,
                              ctx, u, fades)
         y = self.rt.empty(T, self.inner, dtype=f32)
-        ops.linear_scan(u, self.inner + self.gn, self.inner, 0, n, s.state_dim, s.value_dim, "given", None, None, None, "none",
-                        "none", "none", cache[0].state, ctx, y, keep=fades[0], write=fades[1], key_heads=s.groups)
+        first = ops.chunk_scan_first(ctx, self.rt.dtype, s.state_dim, s.value_dim) if self.aligned else None
+        if first != 0:
+            ops.linear_scan(u, self.inner + self.gn, self.inner, 0, n, s.state_dim, s.value_dim, "given", None, None, None, "none",
+                            "none", "none", cache[0].state, ctx, y, keep=fades[0], write=fades[1], key_heads=s.groups,
+                            requests=first)
+        if first is not None:
+            ops.chunk_scan(u, self.inner + self.gn, self.inner, 0, n, s.groups, s.state_dim, s.value_dim, cache[0].state, ctx, y,
+                           first, log_keep=fades[2], write=fades[1])
         out = self.rt.empty(T, self.inner)
         ops.state_space_output(y, proj, x_off, u, self.d, self.norm, n, s.norm_groups, s.eps, s.conv_taps, conv_state, ctx, out)
         return ops.linear(out, self.w_out)
