@@ -426,12 +426,13 @@ __global__ void __launch_bounds__(kThreads) chunk_output_kernel(ChunkArgs a) {
 }
 
 // ------------------------------------------------------------------ operands of a rotated memory
-// From the 32-bit rows of a projection to the rows of the kernels above: q and k turned by the token's
+// From the rows of a projection (32-bit or bfloat16) to the rows of the kernels above: q and k turned by the token's
 // position (pairs (i, i + dims / 2) of the first `dims` channels of every head, angle and rotation in 32-bit), each
 // as a rounded value and a rounded rest, and v rounded: [q | rest of q | k | rest of k | v].
 constexpr int kTurnMaxHalf = 512;
 
-__global__ void __launch_bounds__(256) turn_split_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
+template <typename TP>
+__global__ void __launch_bounds__(256) turn_split_kernel(const TP* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
                                                          int heads, int D, int vv, int dims, const float* __restrict__ inv_freq,
                                                          const int* __restrict__ positions, int first, bf16* __restrict__ rows) {
     __shared__ float cs[kTurnMaxHalf], sn[kTurnMaxHalf];
@@ -441,7 +442,7 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const float* __restrict
     for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &sn[i], &cs[i]);
     __syncthreads();
     lsb_pdl_wait();
-    const float* src = proj + (size_t)t * ld;
+    const TP* src = proj + (size_t)t * ld;
     bf16* dst = rows + (size_t)t * (4 * qk + vv);
     const int pairs = D >> 1, per = 2 * heads * pairs;
     for (int w = threadIdx.x; w < per; w += blockDim.x) {
@@ -450,8 +451,8 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const float* __restrict
         const int hd = (is_q ? hh : hh - heads) * D;
         // the turning pairs first, then the rest two by two
         const int ia = i < half ? i : dims + 2 * (i - half), ib = i < half ? i + half : ia + 1;
-        const float* x = src + (is_q ? q_off : k_off) + hd;
-        float a = x[ia], b = x[ib];
+        const TP* x = src + (is_q ? q_off : k_off) + hd;
+        float a = lsb_to_float(x[ia]), b = lsb_to_float(x[ib]);
         if (i < half) {
             const float u = a * cs[i] - b * sn[i];
             b = b * cs[i] + a * sn[i];
@@ -465,17 +466,18 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const float* __restrict
         o[qk + ib] = __float2bfloat16_rn(b - __bfloat162float(hb));
     }
     for (int w = threadIdx.x * 2; w < vv; w += blockDim.x * 2)
-        *reinterpret_cast<__nv_bfloat162*>(dst + 4 * qk + w) = __floats2bfloat162_rn(src[v_off + w], src[v_off + w + 1]);
+        *reinterpret_cast<__nv_bfloat162*>(dst + 4 * qk + w) = __floats2bfloat162_rn(lsb_to_float(src[v_off + w]), lsb_to_float(src[v_off + w + 1]));
 }
 
 // tokens first .. first + tokens - 1 of the step
-LSB_API int lsb_turn_split(const float* proj, long long ld, int q_off, int k_off, int v_off, int heads, int D, int vv, int dims,
+LSB_API int lsb_turn_split(const void* proj, int dtype, long long ld, int q_off, int k_off, int v_off, int heads, int D, int vv, int dims,
                            const float* inv_freq, const int* positions, int first, int tokens, void* rows, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (heads <= 0 || D <= 0 || D % 2 || vv % 2 || dims < 0 || dims % 2 || dims > D || dims / 2 > kTurnMaxHalf || first < 0)
         return (int)cudaErrorInvalidValue;
-    return lsb_launch(turn_split_kernel, dim3(tokens), dim3(256), 0, stream, 1, proj, ld, q_off, k_off, v_off, heads, D, vv, dims,
-                      inv_freq, positions, first, (bf16*)rows);
+    LSB_DISPATCH_DTYPE(dtype, return lsb_launch(turn_split_kernel<T>, dim3(tokens), dim3(256), 0, stream, 1, (const T*)proj, ld, q_off,
+                                                k_off, v_off, heads, D, vv, dims, inv_freq, positions, first, (bf16*)rows));
+    return 0;
 }
 
 // ------------------------------------------------------------------ host side

@@ -59,9 +59,12 @@ struct RouteOpts {
 
 constexpr int kMaxTop = 32;
 
-// Experts chosen by the token's id: table [rows, top], every choice with the same weight.
+// Experts chosen by the token's id: tables [rows, top], every choice with the same weight.  Several layers'
+// tables are worked through by a launch, a block each, since nothing but the tokens decides.
+constexpr int kMaxTables = 32;
+
 struct TokenRows {
-    const int* table;
+    const int* tables[kMaxTables];
     const int* token_ids;
     int rows;
     float weight;
@@ -192,6 +195,14 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
                  float* __restrict__ row_scale, int* __restrict__ tile_expert,
                  const float* __restrict__ logits, RouteOpts ro, TokenRows by) {
     extern __shared__ int shi[];
+    const int layer = blockIdx.x;
+    ids += (size_t)layer * n;
+    wts += (size_t)layer * n;
+    pos += (size_t)layer * n;
+    row_token += (size_t)layer * cap_tiles * tile;
+    row_scale += (size_t)layer * cap_tiles * tile;
+    tile_expert += (size_t)layer * cap_tiles;
+    const int* table = by.tables[layer];
     int* counts = shi;                  // E
     int* starts = shi + E;              // E + 1, in rows
     lsb_pdl_launch_dependents();
@@ -202,12 +213,12 @@ moe_align_kernel(int* __restrict__ ids, float* __restrict__ wts, int n, int top,
                         threadIdx.x & 31);
         __syncthreads();
     }
-    if (by.table) {                     // no router: a token's experts are its id's row of the table
+    if (table) {                        // no router: a token's experts are its id's row of the table
         for (int i = threadIdx.x; i < n; i += blockDim.x) {
             const int tok = by.token_ids[i / top];
             const bool known = tok >= 0 && tok < by.rows;
             if (!known) lsb_set_status(LSB_BAD_TOKEN);
-            ids[i] = known ? by.table[(size_t)tok * top + i % top] : -1;
+            ids[i] = known ? table[(size_t)tok * top + i % top] : -1;
             wts[i] = by.weight;
         }
         __syncthreads();
@@ -434,21 +445,41 @@ LSB_API int lsb_moe_route(const float* logits, int ld, int n_tokens, int E, int 
                       dim3(32 * warps_per_block), 0, stream, 1, logits, n_tokens, E, top, ro, ids, wts);
 }
 
-// logits given (32-bit [tokens, E]): ids and wts are chosen here first (see lsb_moe_route) and written;
-// table given ([table_rows, top]): they are read from the row of each token's id, the weights all table_weight
+// logits given (32-bit [tokens, E]): ids and wts are chosen here first (see lsb_moe_route) and written
 LSB_API int lsb_moe_align(int* ids, float* wts, int n_tokens, int top, int E, int cap_tiles,
                           int tile, int* pos, int* row_token, float* row_scale, int* tile_expert,
                           const float* logits, int ld, int score, int renorm, const float* bias, int joins, float scale, float eps,
-                          const int* table, const int* token_ids, int table_rows, float table_weight, cudaStream_t stream) {
+                          cudaStream_t stream) {
     const RouteOpts ro = {score, renorm, bias, scale, eps, joins, ld};
-    const TokenRows by = {table, token_ids, table_rows, table_weight};
-    if (table && (logits || !token_ids || table_rows <= 0)) return (int)cudaErrorInvalidValue;
+    const TokenRows by = {};
     if (n_tokens <= 0) return 0;
     const long long n = (long long)n_tokens * top;
     if (E <= 0 || E > 8192 || tile <= 0 || cap_tiles < (n + tile - 1) / tile + E) return (int)cudaErrorInvalidValue;
     if (logits && (top > kMaxTop || top > E || score < 0 || score > 2 || ld < E)) return (int)cudaErrorInvalidValue;
     return lsb_launch(moe_align_kernel, dim3(1), dim3(1024), (size_t)(2 * E + 1) * sizeof(int), stream, 1,
                       ids, wts, (int)n, top, E, cap_tiles, tile, pos, row_token, row_scale, tile_expert, logits, ro, by);
+}
+
+LSB_API int lsb_moe_max_tables() { return kMaxTables; }
+
+// The same for `layers` layers whose experts are named by tables [table_rows, top] of the tokens' ids, each choice with
+// the weight `weight`: every output has a leading dimension of `layers`.
+LSB_API int lsb_moe_align_tables(const int* const* tables, int layers, const int* token_ids, int table_rows, float weight, int* ids,
+                                 float* wts, int n_tokens, int top, int E, int cap_tiles, int tile, int* pos, int* row_token,
+                                 float* row_scale, int* tile_expert, cudaStream_t stream) {
+    if (n_tokens <= 0 || layers <= 0) return 0;
+    const long long n = (long long)n_tokens * top;
+    if (layers > kMaxTables || table_rows <= 0 || top <= 0 || E <= 0 || E > 8192 || tile <= 0 || n > 0x7fffffffLL ||
+        cap_tiles < (n + tile - 1) / tile + E)
+        return (int)cudaErrorInvalidValue;
+    TokenRows by = {};
+    for (int i = 0; i < layers; ++i) by.tables[i] = tables[i];
+    by.token_ids = token_ids;
+    by.rows = table_rows;
+    by.weight = weight;
+    const RouteOpts ro = {};
+    return lsb_launch(moe_align_kernel, dim3(layers), dim3(1024), (size_t)(2 * E + 1) * sizeof(int), stream, 1, ids, wts, (int)n, top, E,
+                      cap_tiles, tile, pos, row_token, row_scale, tile_expert, (const float*)nullptr, ro, by);
 }
 
 // rows[pos[t, k]] = T(wts[t, k] * x[t]): the operand of the grouped tensor-core product, which wants

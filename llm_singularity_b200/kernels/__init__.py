@@ -1021,13 +1021,16 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     (state and out then have ``value_dim + 1`` columns a head, the last one of out being the
     running sum of b dotted with q).  ``q_scale`` multiplies q.  ``key_heads``: heads of q and k, shared by
     groups of ``heads / key_heads`` heads (not with the forget gate).  ``requests``: only the step's first that
-    many, which bring one token each."""
+    many, which bring one token each (``proj`` may end behind them)."""
     _req(proj, "proj", dim=2)
     _req(state, "state", torch.float32, 4)
     _req(out, "out", torch.float32, 2)
     T, ld = proj.shape
     cols = value_dim + (1 if ones else 0)
-    if state.shape[1:] != (heads, cols, key_dim) or out.shape != (T, heads * cols) or ctx.n_tokens != T:
+    if requests is not None and not 0 <= requests <= T:
+        raise KernelError("linear_scan: the requests' single tokens are not in proj")
+    if state.shape[1:] != (heads, cols, key_dim) or out.shape[1] != heads * cols \
+            or (requests is None and (out.shape[0] != T or ctx.n_tokens != T)) or out.shape[0] < (requests or 0):
         raise KernelError("linear_scan: state, out or the step do not fit the sizes")
     key_heads = heads if key_heads is None else key_heads
     if key_heads <= 0 or heads % key_heads or (gate == "forget" and key_heads != heads):
@@ -1039,7 +1042,7 @@ def linear_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: i
     for name, t in (("keep", keep), ("write", write)):
         if t is not None:
             _req(t, name, torch.float32, 2)
-            if t.shape != (T, heads):
+            if t.shape[1] != heads or t.shape[0] < T:
                 raise KernelError(f"linear_scan: {name} must be [tokens, heads]")
     for name, t, n in (("decay", decay, heads), ("f_bias", f_bias, heads * key_dim), ("floor", floor, heads * key_dim)):
         if t is not None:
@@ -1074,10 +1077,11 @@ def turn_heads(proj: torch.Tensor, q_off: int, k_off: int, heads: int, key_dim: 
     _req(inv_freq, "inv_freq", torch.float32, 1)
     T, ld = proj.shape
     dims = 2 * inv_freq.shape[0]
-    if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off) < 0 or max(q_off, k_off) + heads * key_dim > ld:
+    tokens = ctx.n_tokens if tokens is None else tokens
+    if not 0 <= tokens <= T or tokens > ctx.n_tokens or dims > key_dim or min(q_off, k_off) < 0 or max(q_off, k_off) + heads * key_dim > ld:
         raise KernelError("turn_heads: proj, the heads and the step disagree")
     _call("linear_scan", "lsb_turn_heads", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(heads), _i(key_dim), _i(dims),
-          _p(inv_freq), _p(ctx.positions), _i(T if tokens is None else tokens), _stream(proj))
+          _p(inv_freq), _p(ctx.positions), _i(tokens), _stream(proj))
 
 
 # ---------------------------------------- memories that fade by one number per head: prompts on the tensor cores
@@ -1097,17 +1101,17 @@ def chunk_scan_first(ctx, dtype, key_dim: int, value_dim: int) -> Optional[int]:
 
 def turn_split(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, key_dim: int, value_dim: int,
                inv_freq: torch.Tensor, ctx, first: int) -> torch.Tensor:
-    """Rows for ``chunk_scan`` from the 32-bit rows of ``proj``: q and k turned as ``turn_heads`` does, each as a
+    """Rows for ``chunk_scan`` from the rows of ``proj`` (32-bit or bfloat16): q and k turned as ``turn_heads`` does, each as a
     rounded value and a rounded rest, and v rounded: bfloat16 [T, q | rest | k | rest | v], filled from the token
     ``first`` on."""
-    _req(proj, "proj", torch.float32, 2)
+    _req(proj, "proj", dim=2)
     _req(inv_freq, "inv_freq", torch.float32, 1)
     T, ld = proj.shape
     qk, vv, dims = heads * key_dim, heads * value_dim, 2 * inv_freq.shape[0]
     if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off, v_off) < 0 or max(q_off, k_off) + qk > ld or v_off + vv > ld:
         raise KernelError("turn_split: proj, the heads and the step disagree")
     rows = torch.empty(T, 4 * qk + vv, dtype=torch.bfloat16, device=proj.device)
-    _call("chunk_scan", "lsb_turn_split", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(heads), _i(key_dim), _i(vv), _i(dims),
+    _call("chunk_scan", "lsb_turn_split", _p(proj), _i(_dt(proj)), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(heads), _i(key_dim), _i(vv), _i(dims),
           _p(inv_freq), _p(ctx.positions), _i(first), _i(T - first), _p(rows), _stream(proj))
     return rows
 
@@ -1159,16 +1163,17 @@ def chunk_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
 
 
 # ----------------------------------------------------------------- state-space memory
-def state_space_prep(proj: torch.Tensor, x_off: int, dt_off: int, channels: int, conv: torch.Tensor, conv_bias: torch.Tensor,
+def state_space_prep(proj: torch.Tensor, x_off: int, dt: torch.Tensor, channels: int, conv: torch.Tensor, conv_bias: torch.Tensor,
                      dt_bias: torch.Tensor, a_log: torch.Tensor, conv_state: Optional[torch.Tensor], ctx, u: torch.Tensor,
                      fades: torch.Tensor) -> None:
-    """From the 32-bit rows of ``proj``: u [T, channels] = silu(conv_bias + causal convolution of the ``channels``
+    """From the rows of ``proj`` (32-bit or in u's type): u [T, channels] = silu(conv_bias + causal convolution of the ``channels``
     columns from ``x_off`` on), taps ``conv`` [channels, n] whose last column meets the current token, the inputs
-    before a portion from ``conv_state`` [slots, n - 1, channels]; and per head dt = softplus(proj[:, dt_off:] +
-    dt_bias): ``fades`` [3, T, heads] receives exp(-exp(a_log) dt), dt and -exp(a_log) dt.  In a step of single
+    before a portion from ``conv_state`` [slots, n - 1, channels]; and per head dt = softplus(dt + dt_bias)
+    (``dt`` 32-bit [T, heads or more], rows may be strided): ``fades`` [3, T, heads] receives exp(-exp(a_log) dt), dt and -exp(a_log) dt.  In a step of single
     tokens ``conv_state`` is updated here, in others by ``state_space_output``."""
-    _req(proj, "proj", torch.float32, 2)
     _req(u, "u", dim=2)
+    _req(proj, "proj", None if proj.dtype == torch.float32 else u.dtype, 2)
+    _req(dt, "dt", torch.float32, 2, contiguous=False)
     _req(fades, "fades", torch.float32, 3)
     _req(conv, "conv", torch.float32, 2)
     T, ld = proj.shape
@@ -1178,7 +1183,7 @@ def state_space_prep(proj: torch.Tensor, x_off: int, dt_off: int, channels: int,
         if t.shape[0] != k:
             raise KernelError(f"state_space_prep: {name} must have {k} entries")
     if (ctx.n_tokens != T or u.shape != (T, channels) or fades.shape != (3, T, heads) or conv.shape[0] != channels
-            or min(x_off, dt_off) < 0 or x_off + channels > ld or dt_off + heads > ld):
+            or x_off < 0 or x_off + channels > ld or dt.shape[0] != T or dt.shape[1] < heads or dt.stride(1) != 1):
         raise KernelError("state_space_prep: proj, u, the fades and the step do not fit the sizes")
     slots = 1 << 30
     if n > 1:
@@ -1186,7 +1191,7 @@ def state_space_prep(proj: torch.Tensor, x_off: int, dt_off: int, channels: int,
         if conv_state.shape[1:] != (n - 1, channels):
             raise KernelError(f"state_space_prep: conv_state must be [slots, {n - 1}, {channels}]")
         slots = conv_state.shape[0]
-    _call("state_space", "lsb_state_space_prep", _p(proj), _ll(ld), _i(x_off), _i(dt_off), _i(T), _i(channels), _i(heads), _i(n),
+    _call("state_space", "lsb_state_space_prep", _p(proj), _i(_dt(proj)), _ll(ld), _i(x_off), _p(dt), _ll(dt.stride(0)), _i(T), _i(channels), _i(heads), _i(n),
           _p(conv), _p(conv_bias), _p(dt_bias), _p(a_log), _p(conv_state if n > 1 else None), _i(slots), _p(ctx.token_req),
           _p(ctx.q_start), _p(ctx.table_rows), _p(u), _i(_dt(u)), _p(fades[0]), _p(fades[1]), _p(fades[2]),
           _i(1 if ctx.max_q_len == 1 and n > 1 else 0), _stream(u))
@@ -1200,8 +1205,8 @@ def state_space_output(y: torch.Tensor, proj: torch.Tensor, x_off: int, u: torch
     (``groups`` equal parts of the row) times ``weight``.  In steps that bring portions the convolution's inputs in
     ``conv_state`` are replaced by the portions' last ``taps - 1``."""
     _req(y, "y", torch.float32, 2)
-    _req(proj, "proj", torch.float32, 2)
     _req(out, "out", dim=2)
+    _req(proj, "proj", None if proj.dtype == torch.float32 else out.dtype, 2)
     _req(u, "u", out.dtype, 2)
     T, inner = y.shape
     for name, t, k in (("d", d, heads), ("weight", weight, inner)):
@@ -1217,7 +1222,7 @@ def state_space_output(y: torch.Tensor, proj: torch.Tensor, x_off: int, u: torch
         _req(conv_state, "conv_state", torch.float32, 3)
         if conv_state.shape[1:] != (taps - 1, channels):
             raise KernelError(f"state_space_output: conv_state must be [slots, {taps - 1}, {channels}]")
-    _call("state_space", "lsb_state_space_output", _p(y), _p(proj), _ll(proj.shape[1]), _i(x_off), _p(u), _i(channels), _p(d),
+    _call("state_space", "lsb_state_space_output", _p(y), _p(proj), _i(_dt(proj)), _ll(proj.shape[1]), _i(x_off), _p(u), _i(channels), _p(d),
           _p(weight), _i(T), _i(heads), _i(inner // heads), _i(groups), _f(eps), _i(taps if update else 0),
           _p(conv_state if update else None), _i(conv_state.shape[0] if update else 0), _p(ctx.token_req), _p(ctx.q_start),
           _p(ctx.table_rows), _p(out), _i(_dt(out)), _stream(out))
@@ -2113,10 +2118,54 @@ def moe_routed_experts(x: torch.Tensor, logits: torch.Tensor, top: int, score: s
                 gated=gated, add_gate=add_gate)
 
 
+def _expert_tiles(dtype, H: int, F: int, T: int, top: int, E: int):
+    """(tensor cores?, rows of a tile, tiles to set aside) of the experts' grouped products of a step."""
+    tc = MOE_TENSOR_CORES and dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0
+    tile = moe_tile()
+    if tc:
+        mean = T * top / E                  # rows an expert gets
+        tile = MOE_ROW_TILE or (16 if mean <= 8 else 32 if mean <= 16 else 64 if mean <= 32 else 128)
+    return tc, tile, -(-T * top // tile) + E
+
+
+class ExpertPlan:
+    """Which experts a step's tokens go to and where their rows stand, for one layer."""
+    __slots__ = ("ids", "weights", "pos", "row_token", "row_scale", "tile_expert", "tile")
+
+    def __init__(self, ids, weights, pos, row_token, row_scale, tile_expert, tile):
+        self.ids, self.weights, self.pos, self.tile = ids, weights, pos, tile
+        self.row_token, self.row_scale, self.tile_expert = row_token, row_scale, tile_expert
+
+
+def moe_plans(tables, token_ids: torch.Tensor, num_experts: int, dtype, hidden: int, expert_size: int):
+    """A plan for every one of ``tables`` (int32 [R, top], each a layer's: row i names the experts of token id i, all
+    with the weight 1 / top), made by one launch: nothing but the tokens decides."""
+    _req(token_ids, "token_ids", torch.int32, 1)
+    T, E, L = token_ids.shape[0], num_experts, len(tables)
+    R, top = tables[0].shape
+    for t in tables:
+        _req(t, "table", torch.int32, 2)
+        if t.shape != (R, top):
+            raise KernelError("moe_plans: the tables of one launch have one shape")
+    _, tile, cap_tiles = _expert_tiles(dtype, hidden, expert_size, T, top, E)
+    dev, i32 = token_ids.device, torch.int32
+    ids, wts = torch.empty(L, T, top, dtype=i32, device=dev), torch.empty(L, T, top, dtype=torch.float32, device=dev)
+    pos, row_token = torch.empty(L, T * top, dtype=i32, device=dev), torch.empty(L, cap_tiles * tile, dtype=i32, device=dev)
+    row_scale = torch.empty(L, cap_tiles * tile, dtype=torch.float32, device=dev)
+    tile_expert = torch.empty(L, cap_tiles, dtype=i32, device=dev)
+    most = int(_lib("moe").lsb_moe_max_tables())
+    for a in range(0, L, most):
+        n = min(most, L - a)
+        tp = (ctypes.c_void_p * n)(*[_p(t).value for t in tables[a:a + n]])
+        _call("moe", "lsb_moe_align_tables", tp, _i(n), _p(token_ids), _i(R), _f(1.0 / top), _p(ids[a:]), _p(wts[a:]), _i(T), _i(top),
+              _i(E), _i(cap_tiles), _i(tile), _p(pos[a:]), _p(row_token[a:]), _p(row_scale[a:]), _p(tile_expert[a:]), _stream(ids))
+    return [ExpertPlan(ids[i], wts[i], pos[i], row_token[i], row_scale[i], tile_expert[i], tile) for i in range(L)]
+
+
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
                 w_down: torch.Tensor, activation: str, weight_on: str, out: torch.Tensor, route=None,
                 limit: float = 0.0, add: Optional[torch.Tensor] = None, gated: bool = True,
-                add_gate: Optional[torch.Tensor] = None, by_token=None, open_sum: bool = False):
+                add_gate: Optional[torch.Tensor] = None, plan: Optional["ExpertPlan"] = None, open_sum: bool = False):
     """out[t] = sum over k of down_e(act(gate_e u) * up_e u), e = ids[t, k], with u = weights[t, k] * x[t]
     (``weight_on`` "input") or u = x[t] and the sum weighted ("output"); plus ``add[t]`` if given (a shared
     expert's rows, or a callable that makes them: it is called behind the experts' products), in the same
@@ -2124,8 +2173,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
     ``w_gate_up`` [E, 2F, H] has rows alternating gate_i, up_i; ``w_down`` [E, H, F].  ``gated`` False: the
     experts are down_e(act(up_e u)) and ``w_gate_up`` is [E, F, H], the up matrices alone.
 
-    ``by_token = (table, token_ids)``: the experts are those that row ``token_ids[t]`` of the int32 ``table`` [R, top]
-    names, all with the weight 1 / top; ids and weights are filled in.  ``open_sum``: nothing is summed and ``out``
+    ``plan``: the (token, choice) pairs are sorted by expert already (``moe_plans``; ids and weights are the
+    plan's).  ``open_sum``: nothing is summed and ``out``
     may be None; what comes back is (y, pos): the experts' rows and where each (token, choice) has its own."""
     _req(x, "x", dim=2)
     _req(ids, "ids", torch.int32, 2)
@@ -2155,24 +2204,17 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         act = PRODUCT_PLAIN_ACTS[activation]
     # bfloat16 with TMA-friendly sizes: rows gathered in place, two grouped tcgen05 products over
     # 128-row tiles, or over narrow ones where an expert gets a few rows; anything else (32-bit, odd sizes): the plain grouped kernels over 32-row tiles
-    tc = MOE_TENSOR_CORES and x.dtype == torch.bfloat16 and H % 8 == 0 and F % 8 == 0
-    tile = moe_tile()
-    if tc:
-        mean = T * top / E                  # rows an expert gets
-        tile = MOE_ROW_TILE or (16 if mean <= 8 else 32 if mean <= 16 else 64 if mean <= 32 else 128)
-    cap_tiles = -(-T * top // tile) + E
+    tc, tile, cap_tiles = _expert_tiles(x.dtype, H, F, T, top, E)
     dev = x.device
-    table = token_ids = None
-    if by_token is not None:
-        table, token_ids = by_token
-        _req(table, "table", torch.int32, 2)
-        _req(token_ids, "token_ids", torch.int32, 1)
-        if table.shape[1] != top or token_ids.shape[0] != T or route is not None:
-            raise KernelError("moe_experts: the table must have `top` columns, and the step a token id per row")
-    pos = torch.empty(T * top, dtype=torch.int32, device=dev)
-    row_token = torch.empty(cap_tiles * tile, dtype=torch.int32, device=dev)
-    row_scale = torch.empty(cap_tiles * tile, dtype=torch.float32, device=dev)
-    tile_expert = torch.empty(cap_tiles, dtype=torch.int32, device=dev)
+    if plan is not None:
+        if plan.tile != tile or plan.ids.shape != (T, top) or plan.tile_expert.shape[0] != cap_tiles or route is not None:
+            raise KernelError("moe_experts: the plan is another step's")
+        pos, row_token, row_scale, tile_expert = plan.pos, plan.row_token, plan.row_scale, plan.tile_expert
+    else:
+        pos = torch.empty(T * top, dtype=torch.int32, device=dev)
+        row_token = torch.empty(cap_tiles * tile, dtype=torch.int32, device=dev)
+        row_scale = torch.empty(cap_tiles * tile, dtype=torch.float32, device=dev)
+        tile_expert = torch.empty(cap_tiles, dtype=torch.int32, device=dev)
     hidden = torch.empty(cap_tiles * tile, F, dtype=x.dtype, device=dev)
     y = torch.empty(cap_tiles * tile, H, dtype=x.dtype if tc else torch.float32, device=dev)
     s = _stream(x)
@@ -2185,10 +2227,10 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gat
         if route is not None else (None, 0, 0, None, 1.0, 0.0, False)
     if r_logits is not None and (r_logits.shape[0] != T or r_logits.shape[1] < E):
         raise KernelError("moe_experts: the router's logits must be [tokens, experts]")
-    _call("moe", "lsb_moe_align", _p(ids), _p(weights), _i(T), _i(top), _i(E), _i(cap_tiles), _i(tile), _p(pos),
-          _p(row_token), _p(row_scale), _p(tile_expert), _p(r_logits), _i(E if r_logits is None else r_logits.shape[1]),
-          _i(r_score), _i(r_renorm), *_route_options(E, r_bias, r_scale, r_eps, r_joins), _p(table), _p(token_ids),
-          _i(table.shape[0] if table is not None else 0), _f(1.0 / top), s)
+    if plan is None:
+        _call("moe", "lsb_moe_align", _p(ids), _p(weights), _i(T), _i(top), _i(E), _i(cap_tiles), _i(tile), _p(pos),
+              _p(row_token), _p(row_scale), _p(tile_expert), _p(r_logits), _i(E if r_logits is None else r_logits.shape[1]),
+              _i(r_score), _i(r_renorm), *_route_options(E, r_bias, r_scale, r_eps, r_joins), s)
     if tc:
         rows = torch.empty(cap_tiles * tile, H, dtype=x.dtype, device=dev)
         _call("moe", "lsb_moe_gather", _p(x), _i(_dt(x)), _p(pos), _p(weights), _i(on_input), _i(T), _i(top),

@@ -88,6 +88,15 @@ class DecoderModel:
                 part.load(per_owner[path])
         if self.spec.head.tied:
             self.head.tie(self.embedding)
+        groups: Dict[tuple, List[Part]] = {}        # layers whose tokens' ids alone choose the experts plan a step together
+        for part in owners.values():
+            key = part.plan_key() if hasattr(part, "plan_key") else None
+            if key is not None:
+                groups.setdefault(key, []).append(part)
+        for parts in groups.values():
+            tables = [p.table for p in parts]
+            for i, p in enumerate(parts):
+                p.share_plans(tables, i)
         for b in self.blocks:                       # blocks that take per-token inputs from a table
             bind = getattr(b, "bind_embedding", None)    # the embedding holds
             if bind is not None:
@@ -166,6 +175,7 @@ class DecoderModel:
         meets first, the next block's, and may fold it into its last product; such steps are not
         recorded."""
         ops = self.rt.ops
+        ctx.__dict__.pop("expert_plans", None)           # (what a run before this one of the same step made for itself)
         if self.embedding.cache_spec() is not None:      # (its cache id follows the run order's)
             residual = self.embedding.forward(ctx.token_ids, ctx, caches.view(self.spec.num_caches, ctx))
         else:

@@ -14,7 +14,8 @@ with ``shared_gate`` multiplied by the sigmoid of one more 32-bit logit per toke
 stands behind the router's in one matrix.
 
 With ``token_rows`` there is no router: a table of integers, one row per token id, names a token's experts,
-each with the weight 1 / top; the sorting kernel reads it.  A caller that forms the sum over a token's experts
+each with the weight 1 / top; the sorting kernel reads it, for all such layers of a model in one launch a step,
+since nothing but the tokens decides.  A caller that forms the sum over a token's experts
 on its way gets the experts' rows and their places instead (``open_sum``).
 
 The experts' matrices are stacked (``[E, 2F, H]`` with rows alternating gate_i, up_i, and
@@ -92,6 +93,7 @@ class RoutedExperts(Part):
         E, F, H = s.num_experts, s.expert_size, s.hidden_size
         if self.token_rows:
             self.table = tensors["table"].contiguous()
+            self.share_plans([self.table], 0)
             lo, hi = int(self.table.min()), int(self.table.max())
             if lo < 0 or hi >= E:
                 raise ValueError(f"the table of experts holds numbers from {lo} to {hi}, there are {E} experts")
@@ -107,16 +109,32 @@ class RoutedExperts(Part):
         ).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
 
+    # Layers whose experts are named by tables of one shape make their plans together, at the first of them in a
+    # step (the model hands every such part the tables of all of them).
+    def plan_key(self):
+        s = self.spec
+        return (s.token_rows, s.top, s.num_experts, s.hidden_size, s.expert_size) if self.token_rows else None
+
+    def share_plans(self, tables, index: int) -> None:
+        self.tables, self.index = list(tables), index
+
+    def _plan(self, ctx):
+        s = self.spec
+        plans = ctx.__dict__.setdefault("expert_plans", {})
+        key = self.plan_key()
+        if key not in plans:
+            plans[key] = self.rt.ops.moe_plans(self.tables, ctx.token_ids, s.num_experts, self.rt.dtype, s.hidden_size, s.expert_size)
+        return plans[key][self.index]
+
     def forward(self, x, ctx, open_sum: bool = False):
         s, ops, T = self.spec, self.rt.ops, x.shape[0]
         if self.token_rows:
-            ids = self.rt.empty(T, s.top, dtype=torch.int32)
-            weights = self.rt.empty(T, s.top, dtype=torch.float32)
+            plan = self._plan(ctx)
             out = None if open_sum else self.rt.empty(T, s.hidden_size)
             extra = {"limit": float(s.limit)} if s.limit else {}
-            got = ops.moe_experts(x, ids, weights, self.w_gate_up, self.w_down, s.activation, s.weight_on, out, gated=self.gated,
-                                  by_token=(self.table, ctx.token_ids), open_sum=open_sum, **extra)
-            return ExpertRows(got[0], got[1], weights) if open_sum else out
+            got = ops.moe_experts(x, plan.ids, plan.weights, self.w_gate_up, self.w_down, s.activation, s.weight_on, out,
+                                  gated=self.gated, plan=plan, open_sum=open_sum, **extra)
+            return ExpertRows(got[0], got[1], plan.weights) if open_sum else out
         logits = ops.linear(x, self.w_router, out_dtype=torch.float32)
         out = self.rt.empty(T, s.hidden_size)
         extra = {}
