@@ -68,12 +68,8 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
 }
 // two floats as pairs of bfloat16: the rounded values, and the rounded rests
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-    const bf16 ha = __float2bfloat16_rn(a), hb = __float2bfloat16_rn(b);
-    __nv_bfloat162 h;
-    h.x = ha;
-    h.y = hb;
-    hi = *reinterpret_cast<uint32_t*>(&h);
-    lo = pack2(a - __bfloat162float(ha), b - __bfloat162float(hb));
+    hi = pack2(a, b);
+    lo = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 
 // c of every token of the chunk (base-2 logarithm, a pair of floats) and its write factor into shared memory;
@@ -359,19 +355,34 @@ __global__ void __launch_bounds__(kThreads) chunk_output_kernel(ChunkArgs a) {
                 }
             }
         }
-        const float fa = exp2f(ca.x + ca.y) * a.q_scale, fb = exp2f(cb.x + cb.y) * a.q_scale;
+    }
+    // What the chunk's own tokens wrote, sixteen of them at a time up to this warp's.  What came before the warp's
+    // first token fades to it first (one factor per earlier token, and one for the start state) and from there
+    // with the row (one factor at the end): both are at most 1, so nothing overflows on the way.
+    const float2 ref = cum[warp * 16];
+    {
+        const float f = exp2f(ref.x + ref.y);
 #pragma unroll
         for (int j = 0; j < VP / 8; ++j) {
-            o[j][0] *= fa;
-            o[j][1] *= fa;
-            o[j][2] *= fb;
-            o[j][3] *= fb;
+            o[j][0] *= f;
+            o[j][1] *= f;
+            o[j][2] *= f;
+            o[j][3] *= f;
         }
     }
-    // what the chunk's own tokens wrote, sixteen of them at a time up to this warp's
     const uint32_t ka = smem_u32(k_hi + ((i8 >> 1) * 8 + l8) * KS + (i8 & 1) * 8);
     const uint32_t va = smem_u32(vs + ((i8 & 1) * 8 + l8) * VS + (i8 >> 1) * 8);
     for (int g = 0; g <= warp; ++g) {
+        if (g == warp) {
+            const float fa = faded(ca, ref) * a.q_scale, fb = faded(cb, ref) * a.q_scale;
+#pragma unroll
+            for (int j = 0; j < VP / 8; ++j) {
+                o[j][0] *= fa;
+                o[j][1] *= fa;
+                o[j][2] *= fb;
+                o[j][3] *= fb;
+            }
+        }
         float s[2][4];
 #pragma unroll
         for (int j = 0; j < 2; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
@@ -396,9 +407,20 @@ __global__ void __launch_bounds__(kThreads) chunk_output_kernel(ChunkArgs a) {
         for (int j = 0; j < 2; ++j) {
             const int t = g * 16 + j * 8 + 2 * tid4;
             const float2 c0 = cum[t], c1 = cum[t + 1];
-            const float w0 = wr[t] * a.q_scale, w1 = wr[t + 1] * a.q_scale;
-            const float p0 = t <= row_a ? s[j][0] * (faded(ca, c0) * w0) : 0.f, p1 = t + 1 <= row_a ? s[j][1] * (faded(ca, c1) * w1) : 0.f;
-            const float p2 = t <= row_b ? s[j][2] * (faded(cb, c0) * w0) : 0.f, p3 = t + 1 <= row_b ? s[j][3] * (faded(cb, c1) * w1) : 0.f;
+            float p0, p1, p2, p3;
+            if (g < warp) {
+                const float f0 = faded(ref, c0) * wr[t], f1 = faded(ref, c1) * wr[t + 1];
+                p0 = s[j][0] * f0;
+                p1 = s[j][1] * f1;
+                p2 = s[j][2] * f0;
+                p3 = s[j][3] * f1;
+            } else {
+                const float w0 = wr[t] * a.q_scale, w1 = wr[t + 1] * a.q_scale;
+                p0 = t <= row_a ? s[j][0] * (faded(ca, c0) * w0) : 0.f;
+                p1 = t + 1 <= row_a ? s[j][1] * (faded(ca, c1) * w1) : 0.f;
+                p2 = t <= row_b ? s[j][2] * (faded(cb, c0) * w0) : 0.f;
+                p3 = t + 1 <= row_b ? s[j][3] * (faded(cb, c1) * w1) : 0.f;
+            }
             split2(p0, p1, ph[2 * j], pl[2 * j]);
             split2(p2, p3, ph[2 * j + 1], pl[2 * j + 1]);
         }
@@ -426,13 +448,12 @@ __global__ void __launch_bounds__(kThreads) chunk_output_kernel(ChunkArgs a) {
 }
 
 // ------------------------------------------------------------------ operands of a rotated memory
-// From the rows of a projection (32-bit or bfloat16) to the rows of the kernels above: q and k turned by the token's
+// From the 32-bit rows of a projection to the rows of the kernels above: q and k turned by the token's
 // position (pairs (i, i + dims / 2) of the first `dims` channels of every head, angle and rotation in 32-bit), each
 // as a rounded value and a rounded rest, and v rounded: [q | rest of q | k | rest of k | v].
 constexpr int kTurnMaxHalf = 512;
 
-template <typename TP>
-__global__ void __launch_bounds__(256) turn_split_kernel(const TP* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
+__global__ void __launch_bounds__(256) turn_split_kernel(const float* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
                                                          int heads, int D, int vv, int dims, const float* __restrict__ inv_freq,
                                                          const int* __restrict__ positions, int first, bf16* __restrict__ rows) {
     __shared__ float cs[kTurnMaxHalf], sn[kTurnMaxHalf];
@@ -442,7 +463,7 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const TP* __restrict__ 
     for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], &sn[i], &cs[i]);
     __syncthreads();
     lsb_pdl_wait();
-    const TP* src = proj + (size_t)t * ld;
+    const float* src = proj + (size_t)t * ld;
     bf16* dst = rows + (size_t)t * (4 * qk + vv);
     const int pairs = D >> 1, per = 2 * heads * pairs;
     for (int w = threadIdx.x; w < per; w += blockDim.x) {
@@ -451,8 +472,8 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const TP* __restrict__ 
         const int hd = (is_q ? hh : hh - heads) * D;
         // the turning pairs first, then the rest two by two
         const int ia = i < half ? i : dims + 2 * (i - half), ib = i < half ? i + half : ia + 1;
-        const TP* x = src + (is_q ? q_off : k_off) + hd;
-        float a = lsb_to_float(x[ia]), b = lsb_to_float(x[ib]);
+        const float* x = src + (is_q ? q_off : k_off) + hd;
+        float a = x[ia], b = x[ib];
         if (i < half) {
             const float u = a * cs[i] - b * sn[i];
             b = b * cs[i] + a * sn[i];
@@ -466,18 +487,17 @@ __global__ void __launch_bounds__(256) turn_split_kernel(const TP* __restrict__ 
         o[qk + ib] = __float2bfloat16_rn(b - __bfloat162float(hb));
     }
     for (int w = threadIdx.x * 2; w < vv; w += blockDim.x * 2)
-        *reinterpret_cast<__nv_bfloat162*>(dst + 4 * qk + w) = __floats2bfloat162_rn(lsb_to_float(src[v_off + w]), lsb_to_float(src[v_off + w + 1]));
+        *reinterpret_cast<__nv_bfloat162*>(dst + 4 * qk + w) = __floats2bfloat162_rn(src[v_off + w], src[v_off + w + 1]);
 }
 
 // tokens first .. first + tokens - 1 of the step
-LSB_API int lsb_turn_split(const void* proj, int dtype, long long ld, int q_off, int k_off, int v_off, int heads, int D, int vv, int dims,
+LSB_API int lsb_turn_split(const float* proj, long long ld, int q_off, int k_off, int v_off, int heads, int D, int vv, int dims,
                            const float* inv_freq, const int* positions, int first, int tokens, void* rows, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (heads <= 0 || D <= 0 || D % 2 || vv % 2 || dims < 0 || dims % 2 || dims > D || dims / 2 > kTurnMaxHalf || first < 0)
         return (int)cudaErrorInvalidValue;
-    LSB_DISPATCH_DTYPE(dtype, return lsb_launch(turn_split_kernel<T>, dim3(tokens), dim3(256), 0, stream, 1, (const T*)proj, ld, q_off,
-                                                k_off, v_off, heads, D, vv, dims, inv_freq, positions, first, (bf16*)rows));
-    return 0;
+    return lsb_launch(turn_split_kernel, dim3(tokens), dim3(256), 0, stream, 1, proj, ld, q_off, k_off, v_off, heads, D, vv, dims,
+                      inv_freq, positions, first, (bf16*)rows);
 }
 
 // ------------------------------------------------------------------ host side

@@ -368,6 +368,36 @@ __device__ __forceinline__ void epilogue_staged(const GemmParams& prm, unsigned 
     __syncwarp();                                              // the buffer may be refilled right away
 }
 
+// The same for a 32-bit output, COLS columns of the tile in one pass.
+template <int COLS>
+__device__ __forceinline__ void epilogue_staged_f32(const GemmParams& prm, unsigned char* stage_base, uint32_t tmem_base,
+                                                    int q, int lane, int i0, int j0) {
+    constexpr int CPROW = COLS / 4;                           // 16-byte chunks per output row
+    static_assert(CPROW >= 8, "the swizzle needs at least eight chunks per row");
+    uint4* mine = reinterpret_cast<uint4*>(stage_base) + (size_t)q * 32 * CPROW;
+#pragma unroll
+    for (int c0 = 0; c0 < COLS; c0 += 32) {
+        uint32_t r[32];
+        tmem_ld_32x32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)c0, r);
+        tmem_ld_wait();
+        if (prm.plain) plain_act_all(r, prm.plain);
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            mine[lane * CPROW + ((c0 / 4 + k) ^ (lane & 7))] = make_uint4(r[4 * k], r[4 * k + 1], r[4 * k + 2], r[4 * k + 3]);
+    }
+    __syncwarp();
+    float* out = reinterpret_cast<float*>(prm.out);
+#pragma unroll
+    for (int it = 0; it < CPROW; ++it) {
+        const int idx = it * 32 + lane;
+        const int row = idx / CPROW, c = idx % CPROW;
+        const int i = i0 + q * 32 + row;
+        if (i < prm.rows_p)
+            *reinterpret_cast<uint4*>(out + (long long)i * prm.ldc_i + j0 + c * 4) = mine[row * CPROW + (c ^ (row & 7))];
+    }
+    __syncwarp();
+}
+
 // Epilogue of a gated product in the swapped orientation (weights on the tile's 128 rows, gate and up
 // rows alternating; the batch on its BN columns; bfloat16 output [batch, n_out]).  A thread owns one
 // weight row, so an output row of the batch is spread over all 128 threads: written from there it
@@ -630,6 +660,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
 
 // ------------------------------------------------------------------ persistent kernel (prompts)
 // One block per SM walks a list of output tiles (row-major orientation, 128 x BN, one K range).
+// Grouped products (routed experts) walk the same list with the columns fastest, so that a row tile and a
+// group's matrix are shared by blocks that run at the same time; unused row tiles are skipped by every role
+// alike, and nothing is asked for before the list of groups, which a kernel of the step writes, is there.
 // The accumulator is double-buffered in TMEM (2 x BN columns): while the epilogue warps drain
 // tile i from one buffer into global memory, the MMA warp already fills the other with tile i+1,
 // and the TMA warp runs ahead through the ring of stages without regard to tile boundaries.  This
@@ -676,6 +709,9 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
     lsb_pdl_launch_dependents();
     // tile t -> (row block, column block); neighbouring blocks share the weight columns
     const bool weights_p = prm.static_operand == 1;
+    const int* groups = prm.tile_group;
+    auto row_of = [&](int t) { return groups ? t / tiles_n : t % tiles_m; };
+    auto col_of = [&](int t) { return groups ? t % tiles_n : t / tiles_m; };
     int pre = 0;
     if (threadIdx.x == 0) {
         abort_flag = 0;
@@ -686,7 +722,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
         // The weights are not written by anything in the stream: the boxes of the first ring fill are
         // requested at once, before the block meets (tensor memory is being allocated meanwhile) and
         // before the wait on the previous kernel; the activations after it.
-        for (int t = blockIdx.x; t < n_tiles && pre < STAGES; t += gridDim.x) {
+        for (int t = blockIdx.x; t < n_tiles && pre < STAGES && !groups; t += gridDim.x) {
             const int i0 = (t % tiles_m) * kBM, j0 = (t / tiles_m) * BN;
             for (int kb = 0; kb < nkb && pre < STAGES; ++kb, ++pre) {
                 unsigned char* st = stages + (size_t)pre * L::kStageBytes;
@@ -709,7 +745,13 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
             long long it = 0;                                  // K blocks issued so far, over all tiles
             bool ok = true;
             for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
-                const int i0 = (t % tiles_m) * kBM, j0 = (t / tiles_m) * BN;
+                const int i0 = row_of(t) * kBM;
+                int j0 = col_of(t) * BN;
+                if (groups) {
+                    const int g = groups[row_of(t)];
+                    if (g < 0) continue;
+                    j0 += g * prm.group_rows;
+                }
                 for (int kb = 0; kb < nkb; ++kb, ++it) {
                     const int s = (int)(it % STAGES);
                     unsigned char* st = stages + (size_t)s * L::kStageBytes;
@@ -736,7 +778,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
             long long it = 0;
             int local = 0;
             bool ok = true;
-            for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, ++local) {
+            for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
+                if (groups && groups[row_of(t)] < 0) continue;
                 const int a = local & 1;
                 // the epilogue must have drained this accumulator (passes at once the first time)
                 ok = mbar_wait(&acc_empty[a], (uint32_t)((local >> 1) & 1) ^ 1u, &abort_flag);
@@ -756,6 +799,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
                     umma_commit(&empty[s]);
                 }
                 umma_commit(&acc_full[a]);
+                ++local;
             }
         }
     } else {
@@ -763,11 +807,13 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
         const int il = q * 32 + lane;
         const int n_out = prm.swiglu == 1 ? prm.rows_q / 2 : prm.rows_q;
         const bool aligned = !prm.out_f32 && (n_out % 8) == 0 && (((uintptr_t)prm.out) & 15) == 0;
+        const bool aligned32 = prm.out_f32 && !prm.swiglu && (n_out % 4) == 0 && prm.ldc_j == 1 && (((uintptr_t)prm.out) & 15) == 0;
         int local = 0;
         bool ok = true;
-        for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x, ++local) {
+        for (int t = blockIdx.x; t < n_tiles && ok; t += gridDim.x) {
+            if (groups && groups[row_of(t)] < 0) continue;
             const int a = local & 1;
-            const int i0 = (t % tiles_m) * kBM, j0 = (t / tiles_m) * BN;
+            const int i0 = row_of(t) * kBM, j0 = col_of(t) * BN;
             ok = mbar_wait(&acc_full[a], (uint32_t)(local >> 1) & 1, &abort_flag);
             tc_fence_after();
             ok = ok && !abort_flag;
@@ -781,6 +827,10 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
                     else
                         epilogue_staged<kEpiCols, false>(prm, epi, tmem_acc + h * kEpiCols, q, lane, i0, j0 + h * kEpiCols);
                 }
+            } else if (BN >= kEpiCols && aligned32 && j0 + BN <= prm.rows_q) {
+#pragma unroll 1
+                for (int h = 0; h < BN / (kEpiCols / 2); ++h)
+                    epilogue_staged_f32<kEpiCols / 2>(prm, epi, tmem_acc + h * (kEpiCols / 2), q, lane, i0, j0 + h * (kEpiCols / 2));
             } else {
 #pragma unroll 1
                 for (int c0 = 0; c0 < BN; c0 += 32) {
@@ -791,6 +841,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
             }
             tc_fence_before();
             mbar_arrive(&acc_empty[a]);                        // 128 arrivals hand the buffer back
+            ++local;
         }
     }
     tc_fence_before();
@@ -1031,7 +1082,7 @@ LSB_API int lsb_gemm_tc(const void* x, const void* w, void* out, int out_f32, in
         grid.z = splits;
         return launch<256, 4>(mp, mq, prm, grid, stream);
     }
-    if (!swap && !out_f32 && bn >= 128) {
+    if (!swap && !(out_f32 && swiglu) && bn >= 128) {
         // prompts: persistent blocks, double-buffered accumulator
         const int tm = (M + kBM - 1) / kBM, tn = (N + bn - 1) / bn;
         return bn == 256 ? launch_persistent<256, 4>(mp, mq, prm, tm, tn, stream)
@@ -1144,6 +1195,9 @@ LSB_API int lsb_gemm_tc_grouped(const void* x, const void* w, void* out, int out
     switch (bn) {
         case 64: return launch<64, 4>(mp, mq, prm, grid, stream);
         case 128: return launch<128, 6>(mp, mq, prm, grid, stream);
-        default: return launch<256, 4>(mp, mq, prm, grid, stream);
+        default:
+            // (persistent blocks: the tile list is a few times as long as the chip is wide)
+            if (!(out_f32 && swiglu)) return launch_persistent<256, 4>(mp, mq, prm, (int)grid.x, (int)grid.y, stream);
+            return launch<256, 4>(mp, mq, prm, grid, stream);
     }
 }

@@ -1,10 +1,9 @@
 // Around the walk of a state-space memory (S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x): what
 // enters it and what becomes of its read-out.
 //
-//   state_space_prep    per token, from the rows of the wide projection (32-bit, or bfloat16 with dt's columns in
-//                       32-bit rows of their own): a causal convolution per channel over time (x, B and C
-//                       together) with a bias, then silu -> u; and per head dt = softplus(. + dt_bias), the
-//                       fade exp(-exp(A_log) dt) and its logarithm.
+//   state_space_prep    per token, from the 32-bit rows of the wide projection: a causal convolution per
+//                       channel over time (x, B and C together) with a bias, then silu -> u; and per head
+//                       dt = softplus(. + dt_bias), the fade exp(-exp(A_log) dt) and its logarithm.
 //   state_space_output  v = (y + D x) * silu(z); v / sqrt(mean over its norm group of v^2 + eps) * w.
 //
 // The last taps - 1 inputs of the convolution are state, one row per request slot.  They are read by
@@ -19,12 +18,17 @@ LSB_DEFINE_STATUS()
 constexpr int kPrepThreads = 128;
 constexpr int kPrepTokens = 16;          // tokens a thread takes of its channel, one after another (one where a step has few)
 
-__device__ __forceinline__ float ss_silu(float z) { return z / (1.f + expf(-z)); }
+// z / (1 + e^-z).  Where the result is rounded to bfloat16 the special-function unit's exponential and an
+// approximate division (each good to about 1e-7 relative) cost a quarter of the exact ones.
+template <typename T>
+__device__ __forceinline__ float ss_silu(float z) {
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+    else return z / (1.f + expf(-z));
+}
 __device__ __forceinline__ float ss_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 struct PrepArgs {
-    const void* proj; long long ld; int x_off;                 // x | B | C side by side from x_off on
-    const float* dt; long long dt_ld;                           // dt's projection, one column a head
+    const float* proj; long long ld; int x_off, dt_off;         // x | B | C side by side from x_off on; dt, a column a head
     int channels, heads, taps, tokens, tile;
     const float *conv, *conv_bias, *dt_bias, *a_log;            // conv [channels, taps]
     float* conv_state; int n_slots;                             // [slots, taps - 1, channels]
@@ -48,17 +52,16 @@ __device__ __forceinline__ void ss_store4(__nv_bfloat16* p, float a, float b, fl
 }
 
 // W channels a thread (1 or 4), TAPS 2 .. 4 (the inputs of earlier tokens in registers) or 0 (any number).
-template <typename TP, typename T, int W, int TAPS>
+template <typename T, int W, int TAPS>
 __global__ void __launch_bounds__(kPrepThreads) state_space_prep_kernel(PrepArgs a, T* __restrict__ u) {
     lsb_pdl_launch_dependents();
     const int first = blockIdx.y * a.tile, last = min(first + a.tile, a.tokens);
-    const TP* proj = (const TP*)a.proj;
     const int taps = TAPS ? TAPS : a.taps, m = taps - 1;
     if (blockIdx.x == gridDim.x - 1) {                          // the heads' step sizes and fades
         lsb_pdl_wait();
         for (int w = threadIdx.x; w < (last - first) * a.heads; w += kPrepThreads) {
             const int t = first + w / a.heads, h = w % a.heads;
-            const float dt = ss_softplus(a.dt[(size_t)t * a.dt_ld + h] + a.dt_bias[h]);
+            const float dt = ss_softplus(a.proj[(size_t)t * a.ld + a.dt_off + h] + a.dt_bias[h]);
             const float lk = -expf(a.a_log[h]) * dt;
             const size_t at = (size_t)t * a.heads + h;
             a.write[at] = dt;
@@ -80,17 +83,31 @@ __global__ void __launch_bounds__(kPrepThreads) state_space_prep_kernel(PrepArgs
         }
     }
     lsb_pdl_wait();
-    auto load = [&](const auto* p, float (&v)[W]) {
+    auto load = [&](const float* p, float (&v)[W]) {
         if constexpr (W == 4) {
             const float4 x = ss_load4(p);
             v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
         } else {
-            v[0] = lsb_to_float(p[0]);
+            v[0] = p[0];
         }
     };
     int r = -1, t0 = 0, slot = 0;
-    for (int t = first; t < last; ++t) {
-        const int rt = a.token_req[t];
+    constexpr int AHEAD = 8;
+    for (int t8 = first; t8 < last; t8 += AHEAD) {             // eight tokens' inputs in flight together
+    float now8[AHEAD][W];
+    int req8[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        if (t8 + k < last) {
+            req8[k] = a.token_req[t8 + k];
+            load(a.proj + (size_t)(t8 + k) * a.ld + a.x_off + c0, now8[k]);
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        const int t = t8 + k;
+        if (t >= last) break;
+        const int rt = req8[k];
         const bool fresh = rt != r;                             // a request's first token here
         if (fresh) {
             r = rt;
@@ -105,13 +122,15 @@ __global__ void __launch_bounds__(kPrepThreads) state_space_prep_kernel(PrepArgs
         // the input `back` tokens before t, from this portion or from the state
         auto earlier = [&](int back, float (&v)[W]) {
             const int at = t - back;
-            if (at >= t0) load(proj + (size_t)at * a.ld + a.x_off + c0, v);
+            if (at >= t0) load(a.proj + (size_t)at * a.ld + a.x_off + c0, v);
             else load(old + (size_t)(at - t0 + m) * a.channels, v);
         };
         float now[W], acc[W];
-        load(proj + (size_t)t * a.ld + a.x_off + c0, now);
 #pragma unroll
-        for (int w = 0; w < W; ++w) acc[w] = bias[w];
+        for (int w = 0; w < W; ++w) {
+            now[w] = now8[k][w];
+            acc[w] = bias[w];
+        }
         if (TAPS) {
             if (fresh) {
 #pragma unroll
@@ -158,17 +177,18 @@ __global__ void __launch_bounds__(kPrepThreads) state_space_prep_kernel(PrepArgs
         }
         T* dst = u + (size_t)t * a.channels + c0;
         if constexpr (W == 4) {
-            ss_store4(dst, ss_silu(acc[0]), ss_silu(acc[1]), ss_silu(acc[2]), ss_silu(acc[3]));
+            ss_store4(dst, ss_silu<T>(acc[0]), ss_silu<T>(acc[1]), ss_silu<T>(acc[2]), ss_silu<T>(acc[3]));
         } else {
-            dst[0] = lsb_from_float<T>(ss_silu(acc[0]));
+            dst[0] = lsb_from_float<T>(ss_silu<T>(acc[0]));
         }
+    }
     }
 }
 
 struct OutArgs {
     const float* y;                                             // [tokens, heads * V], the walk's read-out
-    const void* proj; long long ld; int x_off;                 // z in the first heads * V columns
-    const float *d, *w;                                         // [heads], [heads * V]
+    const float* proj; long long ld; int x_off;                // z in the first heads * V columns
+    const float *d, *w;                                         // [heads * V] each (d the same for a head's channels)
     int heads, V, groups; float eps;
     int channels, taps;                                         // the convolution's state (taps 0: not updated here)
     float* conv_state; int n_slots;
@@ -176,7 +196,6 @@ struct OutArgs {
 };
 
 // A request's convolution inputs for the next step: its last taps - 1, from the portion and what the state held.
-template <typename TP>
 __device__ __forceinline__ void keep_inputs(const OutArgs& a, size_t t) {
     const int r = a.token_req[t], t0 = a.q_start[r], n = a.q_start[r + 1] - t0, m = a.taps - 1;
     if ((int)t != t0 + n - 1) return;
@@ -189,31 +208,30 @@ __device__ __forceinline__ void keep_inputs(const OutArgs& a, size_t t) {
         float* s = a.conv_state + (size_t)slot * m * a.channels + c;
         for (int j = 0; j < m; ++j) {                           // in order: row j may take what row j + n held
             const int back = m - 1 - j;                         // tokens before the last one
-            s[(size_t)j * a.channels] = back < n ? lsb_to_float(((const TP*)a.proj)[((size_t)t - back) * a.ld + a.x_off + c])
-                                                 : s[(size_t)(j + n) * a.channels];
+            s[(size_t)j * a.channels] = back < n ? a.proj[((size_t)t - back) * a.ld + a.x_off + c] : s[(size_t)(j + n) * a.channels];
         }
     }
 }
 
-constexpr int kOutRegs = 4;
+constexpr int kOutRegs = 2, kOutThreads = 512;
 
 // Block (token, norm group); with taps > 1 one block more per token, which in a request's last token replaces
 // the request's convolution inputs.  Four channels a thread and pass, a group of up to 4,096 channels in
-// registers between the two passes (V a multiple of four: a thread's channels are one head's).
-template <typename TP, typename T>
-__global__ void __launch_bounds__(256) state_space_output_vec_kernel(OutArgs a, const T* __restrict__ u, T* __restrict__ out) {
+// registers between the two passes.
+template <typename T>
+__global__ void __launch_bounds__(kOutThreads, 3) state_space_output_vec_kernel(OutArgs a, const T* __restrict__ u, T* __restrict__ out) {
     __shared__ float scratch[33];
     lsb_pdl_launch_dependents();
     const size_t t = blockIdx.x;
     const int inner = a.heads * a.V, gs = inner / a.groups;
     lsb_pdl_wait();
     if ((int)blockIdx.y == a.groups) {
-        keep_inputs<TP>(a, t);
+        keep_inputs(a, t);
         return;
     }
     const int base = blockIdx.y * gs, step = blockDim.x * 4;
     const float* yr = a.y + t * inner + base;
-    const TP* zr = (const TP*)a.proj + t * a.ld + base;
+    const float* zr = a.proj + t * a.ld + base;
     const T* xr = u + t * a.channels + base;
     float4 v[kOutRegs], z[kOutRegs], x[kOutRegs];
 #pragma unroll
@@ -231,11 +249,11 @@ __global__ void __launch_bounds__(256) state_space_output_vec_kernel(OutArgs a, 
     for (int k = 0; k < kOutRegs; ++k) {
         const int i = threadIdx.x * 4 + k * step;
         if (i < gs) {
-            const float d = a.d[(base + i) / a.V];
-            v[k].x = (v[k].x + d * x[k].x) * ss_silu(z[k].x);
-            v[k].y = (v[k].y + d * x[k].y) * ss_silu(z[k].y);
-            v[k].z = (v[k].z + d * x[k].z) * ss_silu(z[k].z);
-            v[k].w = (v[k].w + d * x[k].w) * ss_silu(z[k].w);
+            const float4 d = ss_load4(a.d + base + i);
+            v[k].x = (v[k].x + d.x * x[k].x) * ss_silu<T>(z[k].x);
+            v[k].y = (v[k].y + d.y * x[k].y) * ss_silu<T>(z[k].y);
+            v[k].z = (v[k].z + d.z * x[k].z) * ss_silu<T>(z[k].z);
+            v[k].w = (v[k].w + d.w * x[k].w) * ss_silu<T>(z[k].w);
             ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
         }
     }
@@ -251,7 +269,7 @@ __global__ void __launch_bounds__(256) state_space_output_vec_kernel(OutArgs a, 
 }
 
 // The same for any sizes.
-template <typename TP, typename T>
+template <typename T>
 __global__ void __launch_bounds__(256) state_space_output_kernel(OutArgs a, const T* __restrict__ u, T* __restrict__ out) {
     extern __shared__ float v_sh[];
     __shared__ float scratch[33];
@@ -260,15 +278,15 @@ __global__ void __launch_bounds__(256) state_space_output_kernel(OutArgs a, cons
     const int inner = a.heads * a.V, gs = inner / a.groups;
     lsb_pdl_wait();
     if ((int)blockIdx.y == a.groups) {
-        keep_inputs<TP>(a, t);
+        keep_inputs(a, t);
         return;
     }
     const int base = blockIdx.y * gs;
     float ss = 0.f;
     for (int i = threadIdx.x; i < gs; i += blockDim.x) {
         const int c = base + i;
-        const float v = (a.y[t * inner + c] + a.d[c / a.V] * lsb_to_float(u[t * a.channels + c])) *
-                        ss_silu(lsb_to_float(((const TP*)a.proj)[t * a.ld + c]));
+        const float v = (a.y[t * inner + c] + a.d[c] * lsb_to_float(u[t * a.channels + c])) *
+                        ss_silu<T>(a.proj[t * a.ld + c]);
         v_sh[i] = v;
         ss += v * v;
     }
@@ -276,19 +294,17 @@ __global__ void __launch_bounds__(256) state_space_output_kernel(OutArgs a, cons
     for (int i = threadIdx.x; i < gs; i += blockDim.x) out[t * inner + base + i] = lsb_from_float<T>(v_sh[i] * inv * a.w[base + i]);
 }
 
-// proj: rows `ld` apart in `proj_dtype`; x | B | C in `channels` columns from x_off on.  dt: 32-bit rows dt_ld
-// apart, `heads` columns.  u [tokens, channels] in `dtype`.  update_state: every request of the step brings one
-// token, and its convolution inputs are replaced here.
-LSB_API int lsb_state_space_prep(const void* proj, int proj_dtype, long long ld, int x_off, const float* dt, long long dt_ld, int tokens,
-                                 int channels, int heads, int taps, const float* conv, const float* conv_bias, const float* dt_bias,
+// proj: 32-bit rows `ld` apart; x | B | C in `channels` columns from x_off on, dt's projection in `heads` columns
+// from dt_off on.  u [tokens, channels] in `dtype`.  update_state: every request of the step brings one token,
+// and its convolution inputs are replaced here.
+LSB_API int lsb_state_space_prep(const float* proj, long long ld, int x_off, int dt_off, int tokens, int channels, int heads, int taps, const float* conv, const float* conv_bias, const float* dt_bias,
                                  const float* a_log, float* conv_state, int n_slots, const int* token_req, const int* q_start,
                                  const int* table_rows, void* u, int dtype, float* keep, float* write, float* log_keep,
                                  int update_state, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (channels <= 0 || heads <= 0 || taps < 1 || (taps > 1 && !conv_state) || (proj_dtype == LSB_BF16 && dtype != LSB_BF16))
-        return (int)cudaErrorInvalidValue;
+    if (channels <= 0 || heads <= 0 || taps < 1 || (taps > 1 && !conv_state)) return (int)cudaErrorInvalidValue;
     PrepArgs a;
-    a.proj = proj; a.ld = ld; a.x_off = x_off; a.dt = dt; a.dt_ld = dt_ld;
+    a.proj = proj; a.ld = ld; a.x_off = x_off; a.dt_off = dt_off;
     a.channels = channels; a.heads = heads; a.taps = taps; a.tokens = tokens;
     a.tile = tokens <= 64 ? 1 : kPrepTokens;
     a.conv = conv; a.conv_bias = conv_bias; a.dt_bias = dt_bias; a.a_log = a_log;
@@ -302,22 +318,17 @@ LSB_API int lsb_state_space_prep(const void* proj, int proj_dtype, long long ld,
     const long long tiles = (tokens + a.tile - 1) / a.tile;
     if (tiles > 65535) return (int)cudaErrorInvalidValue;
     dim3 grid((channels + per_block - 1) / per_block + 1, (unsigned)tiles);
-#define LSB_SS_PREP(TP, W, TAPS) return lsb_launch(state_space_prep_kernel<TP, T, W, TAPS>, grid, dim3(kPrepThreads), 0, stream, 1, a, (T*)u)
-#define LSB_SS_PREP_TAPS(TP, W)                   \
-    do {                                          \
-        if (taps == 4) LSB_SS_PREP(TP, W, 4);     \
-        else if (taps == 3) LSB_SS_PREP(TP, W, 3); \
-        else if (taps == 2) LSB_SS_PREP(TP, W, 2); \
-        else LSB_SS_PREP(TP, W, 0);               \
+#define LSB_SS_PREP(W, TAPS) return lsb_launch(state_space_prep_kernel<T, W, TAPS>, grid, dim3(kPrepThreads), 0, stream, 1, a, (T*)u)
+#define LSB_SS_PREP_TAPS(W)                   \
+    do {                                      \
+        if (taps == 4) LSB_SS_PREP(W, 4);     \
+        else if (taps == 3) LSB_SS_PREP(W, 3); \
+        else if (taps == 2) LSB_SS_PREP(W, 2); \
+        else LSB_SS_PREP(W, 0);               \
     } while (0)
-    if (proj_dtype == LSB_BF16) {
-        using T = __nv_bfloat16;
-        if (vec) LSB_SS_PREP_TAPS(__nv_bfloat16, 4);
-        else LSB_SS_PREP_TAPS(__nv_bfloat16, 1);
-    }
     LSB_DISPATCH_DTYPE(dtype, {
-        if (vec) LSB_SS_PREP_TAPS(float, 4);
-        else LSB_SS_PREP_TAPS(float, 1);
+        if (vec) LSB_SS_PREP_TAPS(4);
+        else LSB_SS_PREP_TAPS(1);
     });
 #undef LSB_SS_PREP_TAPS
 #undef LSB_SS_PREP
@@ -325,14 +336,13 @@ LSB_API int lsb_state_space_prep(const void* proj, int proj_dtype, long long ld,
 }
 
 // taps <= 1: the convolution's state is left alone
-LSB_API int lsb_state_space_output(const float* y, const void* proj, int proj_dtype, long long ld, int x_off, const void* u,
+LSB_API int lsb_state_space_output(const float* y, const float* proj, long long ld, int x_off, const void* u,
                                    int channels, const float* d, const float* w, int tokens, int heads, int V, int groups, float eps,
                                    int taps, float* conv_state, int n_slots, const int* token_req, const int* q_start,
                                    const int* table_rows, void* out, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const int inner = heads * V;
-    if (heads <= 0 || V <= 0 || groups <= 0 || inner % groups || channels < inner || groups >= 65535 ||
-        (proj_dtype == LSB_BF16 && dtype != LSB_BF16))
+    if (heads <= 0 || V <= 0 || groups <= 0 || inner % groups || channels < inner || groups >= 65535)
         return (int)cudaErrorInvalidValue;
     OutArgs a;
     a.y = y; a.proj = proj; a.ld = ld; a.x_off = x_off;
@@ -342,25 +352,19 @@ LSB_API int lsb_state_space_output(const float* y, const void* proj, int proj_dt
     const int gs = inner / groups;
     const size_t smem = (size_t)gs * sizeof(float);
     const bool vec = (uintptr_t)y % 16 == 0 && (uintptr_t)proj % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)u % 16 == 0 &&
-                     (uintptr_t)w % 16 == 0 && ld % 4 == 0 && gs % 4 == 0 && V % 4 == 0 && channels % 4 == 0 && gs <= 1024 * kOutRegs;
+                     (uintptr_t)w % 16 == 0 && ld % 4 == 0 && gs % 4 == 0 && (uintptr_t)d % 16 == 0 && channels % 4 == 0 && gs <= 4 * kOutThreads * kOutRegs;
     if (!vec && smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     int threads = ((gs / (vec ? 4 : 1) + 31) / 32) * 32;
-    threads = threads < 32 ? 32 : threads > 256 ? 256 : threads;
+    const int most = vec ? kOutThreads : 256;
+    threads = threads < 32 ? 32 : threads > most ? most : threads;
     dim3 grid(tokens, groups + (taps > 1 ? 1 : 0));
-#define LSB_SS_OUT(TP)                                                                                              \
-    do {                                                                                                           \
-        if (vec) return lsb_launch(state_space_output_vec_kernel<TP, T>, grid, dim3(threads), 0, stream, 1, a, (const T*)u, (T*)out); \
-        if (smem > 48 * 1024) {                                                                                    \
-            int rc = (int)cudaFuncSetAttribute(state_space_output_kernel<TP, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-            if (rc) return rc;                                                                                     \
-        }                                                                                                          \
-        return lsb_launch(state_space_output_kernel<TP, T>, grid, dim3(threads), smem, stream, 1, a, (const T*)u, (T*)out); \
-    } while (0)
-    if (proj_dtype == LSB_BF16) {
-        using T = __nv_bfloat16;
-        LSB_SS_OUT(__nv_bfloat16);
-    }
-    LSB_DISPATCH_DTYPE(dtype, LSB_SS_OUT(float));
-#undef LSB_SS_OUT
+    LSB_DISPATCH_DTYPE(dtype, {
+        if (vec) return lsb_launch(state_space_output_vec_kernel<T>, grid, dim3(threads), 0, stream, 1, a, (const T*)u, (T*)out);
+        if (smem > 48 * 1024) {
+            int rc = (int)cudaFuncSetAttribute(state_space_output_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+            if (rc) return rc;
+        }
+        return lsb_launch(state_space_output_kernel<T>, grid, dim3(threads), smem, stream, 1, a, (const T*)u, (T*)out);
+    });
     return 0;
 }

@@ -1101,17 +1101,17 @@ def chunk_scan_first(ctx, dtype, key_dim: int, value_dim: int) -> Optional[int]:
 
 def turn_split(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, key_dim: int, value_dim: int,
                inv_freq: torch.Tensor, ctx, first: int) -> torch.Tensor:
-    """Rows for ``chunk_scan`` from the rows of ``proj`` (32-bit or bfloat16): q and k turned as ``turn_heads`` does, each as a
+    """Rows for ``chunk_scan`` from the 32-bit rows of ``proj``: q and k turned as ``turn_heads`` does, each as a
     rounded value and a rounded rest, and v rounded: bfloat16 [T, q | rest | k | rest | v], filled from the token
     ``first`` on."""
-    _req(proj, "proj", dim=2)
+    _req(proj, "proj", torch.float32, 2)
     _req(inv_freq, "inv_freq", torch.float32, 1)
     T, ld = proj.shape
     qk, vv, dims = heads * key_dim, heads * value_dim, 2 * inv_freq.shape[0]
     if ctx.n_tokens != T or dims > key_dim or min(q_off, k_off, v_off) < 0 or max(q_off, k_off) + qk > ld or v_off + vv > ld:
         raise KernelError("turn_split: proj, the heads and the step disagree")
     rows = torch.empty(T, 4 * qk + vv, dtype=torch.bfloat16, device=proj.device)
-    _call("chunk_scan", "lsb_turn_split", _p(proj), _i(_dt(proj)), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(heads), _i(key_dim), _i(vv), _i(dims),
+    _call("chunk_scan", "lsb_turn_split", _p(proj), _ll(ld), _i(q_off), _i(k_off), _i(v_off), _i(heads), _i(key_dim), _i(vv), _i(dims),
           _p(inv_freq), _p(ctx.positions), _i(first), _i(T - first), _p(rows), _stream(proj))
     return rows
 
@@ -1163,17 +1163,16 @@ def chunk_scan(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: in
 
 
 # ----------------------------------------------------------------- state-space memory
-def state_space_prep(proj: torch.Tensor, x_off: int, dt: torch.Tensor, channels: int, conv: torch.Tensor, conv_bias: torch.Tensor,
+def state_space_prep(proj: torch.Tensor, x_off: int, dt_off: int, channels: int, conv: torch.Tensor, conv_bias: torch.Tensor,
                      dt_bias: torch.Tensor, a_log: torch.Tensor, conv_state: Optional[torch.Tensor], ctx, u: torch.Tensor,
                      fades: torch.Tensor) -> None:
-    """From the rows of ``proj`` (32-bit or in u's type): u [T, channels] = silu(conv_bias + causal convolution of the ``channels``
+    """From the 32-bit rows of ``proj``: u [T, channels] = silu(conv_bias + causal convolution of the ``channels``
     columns from ``x_off`` on), taps ``conv`` [channels, n] whose last column meets the current token, the inputs
-    before a portion from ``conv_state`` [slots, n - 1, channels]; and per head dt = softplus(dt + dt_bias)
-    (``dt`` 32-bit [T, heads or more], rows may be strided): ``fades`` [3, T, heads] receives exp(-exp(a_log) dt), dt and -exp(a_log) dt.  In a step of single
+    before a portion from ``conv_state`` [slots, n - 1, channels]; and per head dt = softplus(proj[:, dt_off:] +
+    dt_bias): ``fades`` [3, T, heads] receives exp(-exp(a_log) dt), dt and -exp(a_log) dt.  In a step of single
     tokens ``conv_state`` is updated here, in others by ``state_space_output``."""
     _req(u, "u", dim=2)
-    _req(proj, "proj", None if proj.dtype == torch.float32 else u.dtype, 2)
-    _req(dt, "dt", torch.float32, 2, contiguous=False)
+    _req(proj, "proj", torch.float32, 2)
     _req(fades, "fades", torch.float32, 3)
     _req(conv, "conv", torch.float32, 2)
     T, ld = proj.shape
@@ -1183,7 +1182,7 @@ def state_space_prep(proj: torch.Tensor, x_off: int, dt: torch.Tensor, channels:
         if t.shape[0] != k:
             raise KernelError(f"state_space_prep: {name} must have {k} entries")
     if (ctx.n_tokens != T or u.shape != (T, channels) or fades.shape != (3, T, heads) or conv.shape[0] != channels
-            or x_off < 0 or x_off + channels > ld or dt.shape[0] != T or dt.shape[1] < heads or dt.stride(1) != 1):
+            or min(x_off, dt_off) < 0 or x_off + channels > ld or dt_off + heads > ld):
         raise KernelError("state_space_prep: proj, u, the fades and the step do not fit the sizes")
     slots = 1 << 30
     if n > 1:
@@ -1191,7 +1190,7 @@ def state_space_prep(proj: torch.Tensor, x_off: int, dt: torch.Tensor, channels:
         if conv_state.shape[1:] != (n - 1, channels):
             raise KernelError(f"state_space_prep: conv_state must be [slots, {n - 1}, {channels}]")
         slots = conv_state.shape[0]
-    _call("state_space", "lsb_state_space_prep", _p(proj), _i(_dt(proj)), _ll(ld), _i(x_off), _p(dt), _ll(dt.stride(0)), _i(T), _i(channels), _i(heads), _i(n),
+    _call("state_space", "lsb_state_space_prep", _p(proj), _ll(ld), _i(x_off), _i(dt_off), _i(T), _i(channels), _i(heads), _i(n),
           _p(conv), _p(conv_bias), _p(dt_bias), _p(a_log), _p(conv_state if n > 1 else None), _i(slots), _p(ctx.token_req),
           _p(ctx.q_start), _p(ctx.table_rows), _p(u), _i(_dt(u)), _p(fades[0]), _p(fades[1]), _p(fades[2]),
           _i(1 if ctx.max_q_len == 1 and n > 1 else 0), _stream(u))
@@ -1200,16 +1199,16 @@ def state_space_prep(proj: torch.Tensor, x_off: int, dt: torch.Tensor, channels:
 def state_space_output(y: torch.Tensor, proj: torch.Tensor, x_off: int, u: torch.Tensor, d: torch.Tensor, weight: torch.Tensor,
                        heads: int, groups: int, eps: float, taps: int, conv_state: Optional[torch.Tensor], ctx,
                        out: torch.Tensor) -> None:
-    """v = (y + d[head] * u) * silu(proj's first columns) over the ``heads * V`` columns of ``y`` (32-bit, the walk's
+    """v = (y + d * u) * silu(proj's first columns) over the ``heads * V`` columns of ``y`` (32-bit, the walk's
     read-out; ``u``'s first columns are the convolved x); out = v divided by the root mean square of its part
     (``groups`` equal parts of the row) times ``weight``.  In steps that bring portions the convolution's inputs in
     ``conv_state`` are replaced by the portions' last ``taps - 1``."""
     _req(y, "y", torch.float32, 2)
     _req(out, "out", dim=2)
-    _req(proj, "proj", None if proj.dtype == torch.float32 else out.dtype, 2)
+    _req(proj, "proj", torch.float32, 2)
     _req(u, "u", out.dtype, 2)
     T, inner = y.shape
-    for name, t, k in (("d", d, heads), ("weight", weight, inner)):
+    for name, t, k in (("d", d, inner), ("weight", weight, inner)):
         _req(t, name, torch.float32, 1)
         if t.shape[0] != k:
             raise KernelError(f"state_space_output: {name} must have {k} entries")
@@ -1222,7 +1221,7 @@ def state_space_output(y: torch.Tensor, proj: torch.Tensor, x_off: int, u: torch
         _req(conv_state, "conv_state", torch.float32, 3)
         if conv_state.shape[1:] != (taps - 1, channels):
             raise KernelError(f"state_space_output: conv_state must be [slots, {taps - 1}, {channels}]")
-    _call("state_space", "lsb_state_space_output", _p(y), _p(proj), _i(_dt(proj)), _ll(proj.shape[1]), _i(x_off), _p(u), _i(channels), _p(d),
+    _call("state_space", "lsb_state_space_output", _p(y), _p(proj), _ll(proj.shape[1]), _i(x_off), _p(u), _i(channels), _p(d),
           _p(weight), _i(T), _i(heads), _i(inner // heads), _i(groups), _f(eps), _i(taps if update else 0),
           _p(conv_state if update else None), _i(conv_state.shape[0] if update else 0), _p(ctx.token_req), _p(ctx.q_start),
           _p(ctx.table_rows), _p(out), _i(_dt(out)), _stream(out))

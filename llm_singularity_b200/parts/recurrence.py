@@ -10,9 +10,9 @@ floor that also sets the write strength ("forget": a = floor + (1 - floor) sigmo
 b = 1 - a; no key, no other scale).  The outputs are RMS-normed (all heads together with one weight
 over the row, or each head by itself with one weight of head size or none), optionally multiplied by
 sigmoid or silu of W_g x, and projected by W_o.  With a fixed decay q and k may be rotated by the tokens'
-positions and k scaled (retention): walked tokens leave the projection in 32-bit and are rotated there; prompt
-portions run in chunks on the tensor cores (``csrc/chunk_scan.cu``) with rotated queries and keys as sums of two
-bfloat16 numbers.  Nothing that enters the recurrence is rounded behind its projection.
+positions and k scaled (retention): the projections leave their product in 32-bit, walked tokens are rotated
+there, and prompt portions run in chunks on the tensor cores (``csrc/chunk_scan.cu``) with rotated queries and
+keys as sums of two bfloat16 numbers.
 
 The state starts at zero when a request takes a slot, is 32-bit, and is carried from step to
 step in the slot's row of a ``StateSpec`` cache.  One product makes all projections of a step
@@ -116,22 +116,19 @@ class LinearRecurrence(Part):
     def forward(self, x, ctx, cache, writes_cache: bool = True):
         s, ops = self.spec, self.rt.ops
         o = self.rt.empty(x.shape[0], self.vv, dtype=torch.float32)
-        # prompt portions of a rotated memory in chunks on the tensor cores where they can be, the rest walked
-        first = ops.chunk_scan_first(ctx, self.rt.dtype, s.key_dim, s.value_dim) \
-            if self.position is not None and self.log_decay is not None else None
         # [T, q | k or f | v | g]
-        proj = ops.linear(x, self.w_in) if self.position is None or first is not None \
-            else ops.linear(x, self.w_in, out_dtype=torch.float32)
+        proj = ops.linear(x, self.w_in) if self.position is None else ops.linear(x, self.w_in, out_dtype=torch.float32)
         if self.position is None:
             self._walk(proj, ctx, cache, o)
         else:
+            # prompt portions in chunks on the tensor cores where they can be, the rest walked
+            first = ops.chunk_scan_first(ctx, self.rt.dtype, s.key_dim, s.value_dim) if self.log_decay is not None else None
             if first is None:
                 ops.turn_heads(proj, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx)
                 self._walk(proj, ctx, cache, o)
             elif first:                             # single tokens in front of the portions
-                one = ops.linear(x[:first], self.w_in, out_dtype=torch.float32)
-                ops.turn_heads(one, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx, tokens=first)
-                self._walk(one, ctx, cache, o, requests=first)
+                ops.turn_heads(proj, 0, self.qk, s.num_heads, s.key_dim, self.table[0], ctx, tokens=first)
+                self._walk(proj, ctx, cache, o, requests=first)
             if first is not None:
                 qk = self.qk
                 rows = ops.turn_split(proj, 0, qk, 2 * qk, s.num_heads, s.key_dim, s.value_dim, self.table[0], ctx, first)

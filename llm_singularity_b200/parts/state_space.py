@@ -12,7 +12,7 @@ y times silu(z) is RMS-normed in ``norm_groups`` equal parts with one weight ove
 The walk is the one of linear attention (``csrc/linear_scan.cu``) with C for the query, B for the key, x for the
 value and two numbers per token and head given from outside, exp(-exp(A_log) dt) and dt; prompt portions run
 in chunks on the tensor cores where the sizes allow (``csrc/chunk_scan.cu``).  The projection leaves
-its product in 32-bit (in steps of many tokens only the columns of dt); a kernel in front of the walk convolves and makes the two numbers, a kernel
+its product in 32-bit; a kernel in front of the walk convolves and makes the two numbers, a kernel
 behind it adds D x, gates and norms.  The state S and the convolution's last ``conv_taps - 1`` inputs are
 32-bit ``StateSpec`` rows, zero when a request takes a slot.
 """
@@ -23,9 +23,6 @@ from typing import Dict
 import torch
 
 from .base import CompositeCacheSpec, ParamSpec, Part, StateSpec, register_mixer
-
-
-SPLIT_FROM = 64                 # steps of more tokens than this make the wide projection and the step sizes' as two products
 
 
 @register_mixer("state_space")
@@ -61,13 +58,11 @@ class StateSpace(Part):
         w = tensors["in"]
         pad = -w.shape[0] % 8                       # rows of the product start on 16-byte boundaries: the columns behind dt are zero
         self.w_in = (torch.cat([w, w.new_zeros(pad, w.shape[1])]) if pad else w).contiguous()
-        wide = self.inner + self.channels
-        self.w_wide, self.w_dt = self.w_in[:wide], self.w_in[wide:]           # (views: rows of one matrix)
-        self.two_products = self.rt.dtype == torch.bfloat16 and wide % 8 == 0 and w.shape[1] % 8 == 0
         self.w_out = tensors["o"].contiguous()
         self.conv, self.conv_bias = tensors["conv"].contiguous(), tensors["conv_bias"].contiguous()
         self.dt_bias, self.a_log, self.d = (tensors[n].contiguous() for n in ("dt_bias", "A_log", "D"))
         self.norm = tensors["norm"].contiguous()
+        self.skip = self.d.repeat_interleave(self.spec.value_dim).contiguous()        # (one number per channel, as the kernel reads it)
 
     def cache_spec(self):
         s = self.spec
@@ -80,16 +75,11 @@ class StateSpace(Part):
         s, ops = self.spec, self.rt.ops
         T, n, f32 = x.shape[0], s.num_heads, torch.float32
         x_off, dt_off = self.inner, self.inner + self.channels
-        if self.two_products and T > SPLIT_FROM:
-            # many rows: the wide columns leave in the compute dtype, the step sizes in 32-bit
-            proj, dt = ops.linear(x, self.w_wide), ops.linear(x, self.w_dt, out_dtype=f32)
-        else:
-            proj = ops.linear(x, self.w_in, out_dtype=f32)                    # [T, z | x | B | C | dt]
-            dt = proj[:, dt_off:]
+        proj = ops.linear(x, self.w_in, out_dtype=f32)                        # [T, z | x | B | C | dt]
         u = self.rt.empty(T, self.channels)                                  # [T, x | B | C] convolved
         fades = self.rt.empty(3, T, n, dtype=f32)                            # keep, write, log keep
         conv_state = cache[1].state if s.conv_taps > 1 else None
-        ops.state_space_prep(proj, x_off, dt, self.channels, self.conv, self.conv_bias, self.dt_bias, self.a_log, conv_state,
+        ops.state_space_prep(proj, x_off, dt_off, self.channels, self.conv, self.conv_bias, self.dt_bias, self.a_log, conv_state,
                              ctx, u, fades)
         y = self.rt.empty(T, self.inner, dtype=f32)
         first = ops.chunk_scan_first(ctx, self.rt.dtype, s.state_dim, s.value_dim) if self.aligned else None
@@ -101,5 +91,5 @@ class StateSpace(Part):
             ops.chunk_scan(u, self.inner + self.gn, self.inner, 0, n, s.groups, s.state_dim, s.value_dim, cache[0].state, ctx, y,
                            first, log_keep=fades[2], write=fades[1])
         out = self.rt.empty(T, self.inner)
-        ops.state_space_output(y, proj, x_off, u, self.d, self.norm, n, s.norm_groups, s.eps, s.conv_taps, conv_state, ctx, out)
+        ops.state_space_output(y, proj, x_off, u, self.skip, self.norm, n, s.norm_groups, s.eps, s.conv_taps, conv_state, ctx, out)
         return ops.linear(out, self.w_out)
